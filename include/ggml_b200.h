@@ -41,6 +41,7 @@ enum b200_type {
     B200_TYPE_Q8_K = 15,
     B200_TYPE_I32 = 26,
     B200_TYPE_I64 = 27,
+    B200_TYPE_BF16 = 30,
     B200_TYPE_MXFP4 = 39,
 };
 

@@ -43,6 +43,36 @@ enum {
  * r * n_local; src[1] is a scratch tensor of the node's size. */
 enum { B200_OP_TP_ALL_REDUCE = 0x4200, B200_OP_TP_ALL_GATHER = 0x4201 };
 
+/* Ops outside ggml's enum for decoders with dense weights, recurrent layers and latent attention (arch_rukusun.cpp emits them;
+ * every constant is a parameter of the node).  "F32 / BF16" below: rows of either type.  f: the op_params word holds the bits
+ * of a float.  A step's sequences: `seg` I32 [8, n_seg] = {first row, rows, state slot, starts from nothing, position of the
+ * first row, first entry in tab, position of that entry, -}; `row_seg` I32 [n] the sequence of every row; `tab` I32 [n_tab]
+ * the cells of the sequences' positions one after the other; `pos` I32 [n].
+ *
+ * DENSE_MM       w [k, n] F32 / BF16, x [k, m] F32 / BF16, addend [n, m] F32 or null, norm weight [k] F32 or null -> [n, m] F32 /
+ *                BF16: y = act(w (x / rms(x) * norm)) + addend.  op_params: 0 act (0 none, 1 tanh-form gelu), 1 f eps.
+ * RMS_NORM_W     x F32 rows, weight [ne0] F32 -> F32 / BF16 rows.  op_params: 0 f eps.
+ * TAKE_ROWS      table F32 / BF16, ids I32 -> F32 / BF16 rows times a factor.  op_params: 0 f factor.
+ * GLA            gated linear attention of every head, its output normed per head and gated: proj F32 [., n] with q, k, v, g and
+ *                the low-rank decay input at element offsets; src 1 decay weight [rank, heads dim], 2 decay bias F32, 3 norm
+ *                weight [vdim] F32, 4 state F32 [heads dim vdim, slots] (read and updated), 5 seg, 6 scratch F32 (null: token
+ *                by token) -> F32 / BF16 [heads vdim, n].  op_params: 0 heads, 1 dim, 2 vdim, 3..7 offsets of q, k, v, g, decay
+ *                input, 8 f factor of q, 9 f 1 / tau, 10 f eps, 11 n_seg bound of rows per sequence, 12 rank.
+ * Latent attention, op_params: 0 heads, 1 dim, 2 rot, 3 rank of the latent, 4 vdim, 5 window (0: none), 6 f score factor, 7 f eps,
+ *                8 f rotary base, 9 rotary dims, 10..12 offsets of q, latent and gate in proj, 13 keys per split, 14 splits.
+ *                A cell's row holds the normed latent, then the rotated key part.  ukv [rank, heads (dim + vdim)]: key rows, then
+ *                value rows.
+ * LATENT_STORE   proj, pos, norm weight [rank] F32, cells I32 [n] -> aliases the cell rows it writes.
+ * LATENT_QUERY   proj, pos, norm weight, cells, ukv, cell rows (written as by STORE) -> F32 [rank + rot, heads, n]: queries taken
+ *                through the key weight, and rotated.
+ * LATENT_DECODE  queries, pos, cell rows, row_seg, seg, tab -> F32 [rank + 2, heads, splits, n]: per split the weighted sum of
+ *                latents, running maximum, sum of weights.
+ * LATENT_VALUE   those, pos, ukv, proj, sink [heads] F32 -> F32 / BF16 [heads vdim, n]: splits merged, the value weight, the gate.
+ * LATENT_ATTN    proj, pos, kv [heads (dim + vdim), n_tab], latent rows by tab entry, sink, seg -> F32 / BF16 [heads vdim, n]. */
+enum { B200_OP_DENSE_MM = 0x4210, B200_OP_RMS_NORM_W = 0x4211, B200_OP_TAKE_ROWS = 0x4212, B200_OP_GLA = 0x4213,
+       B200_OP_LATENT_STORE = 0x4214, B200_OP_LATENT_QUERY = 0x4215, B200_OP_LATENT_DECODE = 0x4216, B200_OP_LATENT_VALUE = 0x4217,
+       B200_OP_LATENT_ATTN = 0x4218 };
+
 /* enum ggml_unary_op value carried in op_params[0] of a GGML_OP_UNARY node (crates/ggml/src/ops.rs:1632-1636) */
 enum { GGML_UNARY_OP_SILU = 10 };
 

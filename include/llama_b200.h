@@ -91,6 +91,21 @@ int b200_llama_load_gguf_tp(const char *path, int device, int32_t n_ctx, int32_t
                             int32_t tp_size, const void *id128, b200_llama **out);
 int b200_llama_get_hparams(const b200_llama *ctx, struct b200_llama_hparams *out);
 
+/* ---- models described by a configuration file --------------------------------------------------------------
+ * Architectures other than llama come as a folder with config.json and model.safetensors; config.json's "architecture"
+ * picks one of the library's (Rukusun).  dtype: what the weight matrices are kept in, B200_TYPE_BF16 (matrix products with
+ * BF16 operands and F32 sums; norms, recurrences, scores and the residual stream in F32) or B200_TYPE_F32 (everything in
+ * F32).  n_seq: sequences alive at a time (state slots).  b200_model_load_dir loads the folder; b200_model_new makes the
+ * context of a configuration (the text of a config.json) whose tensors b200_llama_set_tensor then sets under their names in the
+ * file, F32 or BF16, in any order once the tensors that only a shape describes are announced with b200_llama_learn_shape.
+ * Decode calls are the same as for llama; these architectures want a sequence's tokens together and in order. */
+int b200_model_new(const char *config_json, int dtype, int device, int32_t n_ctx, int32_t n_batch, int32_t n_seq, b200_llama **out);
+int b200_model_load_dir(const char *dir, int dtype, int device, int32_t n_ctx, int32_t n_batch, int32_t n_seq, b200_llama **out);
+int b200_llama_learn_shape(b200_llama *ctx, const char *name, int64_t ne0, int64_t ne1);
+int32_t b200_llama_n_vocab(const b200_llama *ctx);
+const char *b200_llama_arch_name(const b200_llama *ctx);
+int32_t b200_llama_n_tensors(const b200_llama *ctx);
+
 /* One model tensor under its GGUF name (crates/llama/src/model.rs: token_embd.weight, output_norm.weight,
  * output.weight, blk.N.{attn_norm,attn_q,attn_k,attn_v,attn_output,ffn_norm,ffn_gate,ffn_up,ffn_down}.weight).
  * data: ggml blocks of `type`, ne1 rows of ne0 elements, in host memory.  output.weight may be left out
@@ -114,6 +129,8 @@ int b200_llama_decode_seqs(b200_llama *ctx, const int32_t *tokens, const int32_t
 
 /* Forget every cached position (DecodeContext::kv_clear). */
 int b200_llama_kv_clear(b200_llama *ctx);
+/* Forget one sequence: its cells and its state slot are free for others (llama_memory_seq_rm over a whole sequence). */
+int b200_llama_seq_rm(b200_llama *ctx, int32_t seq);
 /* Cells in use, and the padded cell count the next step's attention would span. */
 int32_t b200_llama_kv_used(const b200_llama *ctx);
 

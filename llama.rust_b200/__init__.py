@@ -17,7 +17,7 @@ import numpy as np
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libggml-b200.so")
 
-F32, F16, Q4_0, Q8_0, Q4_K, Q6_K, Q8_K, MXFP4 = 0, 1, 2, 8, 12, 14, 15, 39
+F32, F16, Q4_0, Q8_0, Q4_K, Q6_K, Q8_K, BF16, MXFP4 = 0, 1, 2, 8, 12, 14, 15, 30, 39
 ACT_Q8_0, ACT_Q8_K, ACT_Q8_K_4X8, ACT_Q8_K_MIXED = 1, 2, 3, 4
 ROUTE_AUTO, ROUTE_ROWDOT, ROUTE_REPACK, ROUTE_TILED = 0, 1, 2, 3
 STATUS_SUCCESS = 0

@@ -4,6 +4,7 @@
 
 The library is plain CUDA C++ behind a C ABI; nothing here needs PyTorch.
 """
+import fcntl
 import glob
 import os
 import subprocess
@@ -40,7 +41,8 @@ def build(verbose=False, force=False):
     if not force and up_to_date():
         return OUT
     nvcc = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
-    cmd = [nvcc] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-o", OUT] + sources()
+    part = f"{OUT}.{os.getpid()}.part"
+    cmd = [nvcc] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-o", part] + sources()
     env = dict(os.environ)
     env.pop("CXX", None)
     env.pop("CC", None)
@@ -48,8 +50,20 @@ def build(verbose=False, force=False):
     if verbose or r.returncode != 0:
         sys.stderr.write(r.stdout + r.stderr)
     if r.returncode != 0:
+        if os.path.exists(part):
+            os.unlink(part)
         raise RuntimeError("nvcc failed building libggml-b200.so")
+    os.replace(part, OUT)
     return OUT
+
+
+def ensure():
+    """the library, built by the first of several processes that want it (the command-line programs call this)"""
+    if up_to_date():
+        return OUT
+    with open(OUT + ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build()
 
 
 if __name__ == "__main__":

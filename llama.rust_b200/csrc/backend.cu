@@ -7,6 +7,7 @@
 // in a buffer of this backend are kept in the 32-row tile layout: set_tensor re-orders the ggml blocks
 // on the way in, get_tensor on the way out, get_alloc_size reports the padded size.
 #include <algorithm>
+#include <cmath>
 #include <cstdio>
 #include <cstring>
 #include <mutex>
@@ -27,7 +28,7 @@ struct TypeTraits { int blck; int size; };
 static TypeTraits traits(int type) {
     switch (type) {
         case B200_TYPE_F32: return {1, 4};
-        case B200_TYPE_F16: return {1, 2};
+        case B200_TYPE_F16: case B200_TYPE_BF16: return {1, 2};
         case B200_TYPE_Q4_0: return {32, 18};
         case B200_TYPE_Q8_0: return {32, 34};
         case B200_TYPE_Q4_K: return {256, 144};
@@ -143,7 +144,7 @@ struct BackendCtx {
 };
 constexpr size_t SHADOW_MAX_BYTES = 1 << 20;
 constexpr int64_t ROPE_TABLE_MIN_ROWS = 4096, ROPE_TABLE_MAX_ROWS = 1 << 20;
-constexpr size_t ROPE_TABLES_KEPT = 4, GRAPHS_KEPT = 512;   // a tensor-parallel step is ~2 node lists per layer
+constexpr size_t ROPE_TABLES_KEPT = 64, GRAPHS_KEPT = 512;   // a tensor-parallel step is ~2 node lists per layer
 
 static std::mutex g_mu;
 static std::vector<ggml_backend_device *> g_devices;
@@ -426,8 +427,88 @@ static bool supports_tp(const ggml_tensor *op, std::string *why) {
     return true;
 }
 
+// ---- ops of decoders with dense weights (B200_OP_DENSE_MM and the ones after it) ---------------------------------
+static bool dense_rows(const ggml_tensor *t) {   // F32 / BF16 rows, dense inside, stacked on dim 1
+    if (!t || (t->type != B200_TYPE_F32 && t->type != B200_TYPE_BF16)) return false;
+    const size_t es = t->type == B200_TYPE_F32 ? 4 : 2;
+    return t->nb[0] == es && t->nb[1] % es == 0 && t->ne[2] == 1 && t->ne[3] == 1;
+}
+static int64_t row_ld(const ggml_tensor *t) { return (int64_t)(t->nb[1] / t->nb[0]); }
+static bool i32_list(const ggml_tensor *t, int64_t at_least) {
+    return t && t->type == B200_TYPE_I32 && is_contiguous(t) && t->ne[0] * t->ne[1] >= at_least;
+}
+static bool f32_vec(const ggml_tensor *t, int64_t n) { return t && t->type == B200_TYPE_F32 && t->nb[0] == 4 && t->ne[0] >= n; }
+
+static bool supports_dense(const ggml_tensor *op, std::string *why) {
+    auto no = [&](const char *m) { if (why) *why = m; return false; };
+    const ggml_tensor *a = op->src[0], *b = op->src[1];
+    const int32_t *p = op->op_params;
+    switch (op->op) {
+        case B200_OP_DENSE_MM:
+            if (!dense_rows(a) || !is_contiguous(a) || !dense_rows(b) || !dense_rows(op)) return no("dense mat-mul wants F32 / BF16 rows");
+            if (a->ne[0] != b->ne[0] || op->ne[0] != a->ne[1] || op->ne[1] != b->ne[1]) return no("dense mat-mul: shape");
+            if (op->src[2] && (!dense_rows(op->src[2]) || op->src[2]->type != B200_TYPE_F32 || op->src[2]->ne[0] != op->ne[0] || op->src[2]->ne[1] != op->ne[1]))
+                return no("dense mat-mul: the addend must be F32 of the result's shape");
+            if (op->src[3] && (!f32_vec(op->src[3], a->ne[0]) || b->type != B200_TYPE_F32 || b->ne[1] > DENSE_FEW_ROWS)) return no("dense mat-mul: norm weight");
+            return p[0] == 0 || p[0] == 1 ? true : no("dense mat-mul: activation function");
+        case B200_OP_RMS_NORM_W:
+            if (!dense_rows(a) || a->type != B200_TYPE_F32 || !dense_rows(op) || !same_shape(a, op) || !f32_vec(b, a->ne[0])) return no("rms_norm_w wants F32 rows");
+            return true;
+        case B200_OP_TAKE_ROWS:
+            if (!dense_rows(a) || !i32_list(b, op->ne[1]) || !dense_rows(op) || op->ne[0] != a->ne[0]) return no("take_rows wants F32 / BF16 rows and I32 ids");
+            return true;
+        case B200_OP_GLA: {
+            const int64_t H = p[0], d = p[1], e = p[2], R = p[12];
+            if (!dense_rows(a) || a->type != B200_TYPE_F32 || !dense_rows(op)) return no("gla wants F32 rows");
+            if (H <= 0 || d <= 0 || e <= 0 || R <= 0 || op->ne[0] != H * e || op->ne[1] != a->ne[1]) return no("gla: shape");
+            if (p[3] < 0 || p[3] + H * d > a->ne[0] || p[4] < 0 || p[4] + H * d > a->ne[0] || p[5] < 0 || p[5] + H * e > a->ne[0] || p[6] < 0 ||
+                p[6] + H * e > a->ne[0] || p[7] < 0 || p[7] + R > a->ne[0])
+                return no("gla: an operand lies outside the projection's rows");
+            if (!dense_rows(b) || !is_contiguous(b) || b->ne[0] != R || b->ne[1] != H * d || !f32_vec(op->src[2], H * d) || !f32_vec(op->src[3], e)) return no("gla: weights");
+            if (!dense_rows(op->src[4]) || op->src[4]->type != B200_TYPE_F32 || op->src[4]->ne[0] != H * d * e || !is_contiguous(op->src[4])) return no("gla: state");
+            if (!i32_list(op->src[5], 8) || op->src[5]->ne[0] != 8) return no("gla: segments");
+            if (op->src[6] && !f32_vec(op->src[6], (int64_t)gla_scratch_floats(H, d, e, a->ne[1], op->src[5]->ne[1]))) return no("gla: scratch");
+            return true;
+        }
+        default: break;
+    }
+    // latent attention
+    const int64_t H = p[0], d = p[1], rot = p[2], R = p[3], e = p[4];
+    if (H <= 0 || d <= 0 || rot < 0 || R <= 0 || e <= 0 || p[9] < 0 || p[9] % 2 || p[9] > rot) return no("latent attention: parameters");
+    const ggml_tensor *proj = op->op == B200_OP_LATENT_VALUE ? op->src[3] : op->op == B200_OP_LATENT_DECODE ? nullptr : a;
+    if (proj && (!dense_rows(proj) || proj->type != B200_TYPE_F32 || p[10] < 0 || p[10] + H * (d + rot) > proj->ne[0] || p[11] < 0 || p[11] + R + rot > proj->ne[0] ||
+                 p[12] < 0 || p[12] + H > proj->ne[0]))
+        return no("latent attention: projection rows");
+    const int64_t n = proj ? proj->ne[1] : a ? a->ne[2] : 0;
+    if (n <= 0 || !i32_list(b, n)) return no("latent attention: positions");
+    const auto cell_rows = [&](const ggml_tensor *t) { return dense_rows(t) && t->ne[0] >= R + rot && t->nb[1] % 16 == 0; };
+    const auto up = [&](const ggml_tensor *t) { return dense_rows(t) && is_contiguous(t) && t->ne[0] == R && t->ne[1] == H * (d + e); };
+    switch (op->op) {
+        case B200_OP_LATENT_STORE:
+            return f32_vec(op->src[2], R) && i32_list(op->src[3], n) && cell_rows(op) ? true : no("latent store: operands");
+        case B200_OP_LATENT_QUERY:
+            return f32_vec(op->src[2], R) && i32_list(op->src[3], n) && up(op->src[4]) && cell_rows(op->src[5]) && op->src[5]->type == op->src[4]->type &&
+                           dense_f32(op) && op->ne[0] == R + rot && op->ne[1] == H && op->ne[2] == n ? true : no("latent query: operands");
+        case B200_OP_LATENT_DECODE:
+            return dense_f32(a) && a->ne[0] == R + rot && a->ne[1] == H && cell_rows(op->src[2]) && i32_list(op->src[3], n) && i32_list(op->src[4], 8) &&
+                           i32_list(op->src[5], 1) && dense_f32(op) && op->ne[0] == (R + 2) * H && op->ne[1] == p[14] && op->ne[2] == n && p[13] > 0 ? true : no("latent decode: operands");
+        case B200_OP_LATENT_VALUE:
+            return dense_f32(a) && a->ne[0] == (R + 2) * H && a->ne[1] == p[14] && a->ne[2] == n && up(op->src[2]) && f32_vec(op->src[4], H) && dense_rows(op) &&
+                           op->ne[0] == H * e && op->ne[1] == n && p[13] > 0 ? true : no("latent value: operands");
+        case B200_OP_LATENT_ATTN: {
+            const ggml_tensor *kv = op->src[2], *rows = op->src[3];
+            return dense_rows(kv) && kv->ne[0] == H * (d + e) && dense_rows(rows) && rows->ne[0] >= R + rot && rows->ne[1] == kv->ne[1] && rows->type == kv->type &&
+                           f32_vec(op->src[4], H) && i32_list(op->src[5], 8) && dense_rows(op) && op->ne[0] == H * e && op->ne[1] == n ? true : no("latent attention: operands");
+        }
+        default: return no("unknown op");
+    }
+}
+
 static bool op_supported(const ggml_tensor *op, std::string *why) {
     switch (op->op) {
+        case B200_OP_DENSE_MM: case B200_OP_RMS_NORM_W: case B200_OP_TAKE_ROWS: case B200_OP_GLA: case B200_OP_LATENT_STORE: case B200_OP_LATENT_QUERY:
+        case B200_OP_LATENT_DECODE: case B200_OP_LATENT_VALUE: case B200_OP_LATENT_ATTN:
+            return supports_dense(op, why);
         case B200_OP_TP_ALL_REDUCE: case B200_OP_TP_ALL_GATHER: return supports_tp(op, why);
         case GGML_OP_NONE: case GGML_OP_RESHAPE: case GGML_OP_VIEW: case GGML_OP_PERMUTE: case GGML_OP_TRANSPOSE:
             return true;
@@ -779,20 +860,9 @@ static int rope_fill_host(BackendCtx *bc, const ggml_tensor *op, const int32_t *
                            bc->rope_host.data());
 }
 
-// Before a node list is issued: every ROPE node's by-position table exists and reaches its largest
-// position.  All device work this needs (allocation, upload) happens here, outside any capture.
-static int rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
-    std::vector<int32_t> p;
-    std::vector<float> factors;
-    int rc = rope_positions(bc, op, &p);
-    if (rc == B200_STATUS_SUCCESS) rc = rope_factors(bc, op, &factors);
-    if (rc != B200_STATUS_SUCCESS || p.empty()) return rc;
-    const int32_t pmin = *std::min_element(p.begin(), p.end()), pmax = *std::max_element(p.begin(), p.end());
-    if (pmin < 0 || pmax >= ROPE_TABLE_MAX_ROWS) {
-        bc->capturable = false;   // served by the per-token table, built while the node is issued
-        return B200_STATUS_SUCCESS;
-    }
-    const std::vector<int32_t> key = rope_param_key(op, factors);
+// The table of a parameter set, reaching position pmax; fill puts the rows of the positions it is given into bc->rope_host.
+template <typename Fill>
+static int rope_reserve(BackendCtx *bc, const std::vector<int32_t> &key, int32_t pmax, Fill fill) {
     BackendCtx::RopeTable *t = nullptr;
     for (auto &cand : bc->rope_by_pos)
         if (cand.key == key) t = &cand;
@@ -817,7 +887,7 @@ static int rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
     while (rows <= pmax) rows *= 2;
     std::vector<int32_t> all(rows);
     for (int64_t i = 0; i < rows; i++) all[i] = (int32_t)i;
-    rc = rope_fill_host(bc, op, all.data(), rows, factors);
+    int rc = fill(all);
     if (rc != B200_STATUS_SUCCESS) return rc;
     B200_CUDA(cudaStreamSynchronize(bc->stream));   // launches in flight may still read the smaller table
     if (t->dev) B200_CUDA(cudaFree(t->dev));
@@ -829,6 +899,24 @@ static int rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
     t->rows = rows;
     t->used = ++bc->rope_clock;
     return B200_STATUS_SUCCESS;
+}
+
+// Before a node list is issued: every ROPE node's by-position table exists and reaches its largest
+// position.  All device work this needs (allocation, upload) happens here, outside any capture.
+static int rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
+    std::vector<int32_t> p;
+    std::vector<float> factors;
+    int rc = rope_positions(bc, op, &p);
+    if (rc == B200_STATUS_SUCCESS) rc = rope_factors(bc, op, &factors);
+    if (rc != B200_STATUS_SUCCESS || p.empty()) return rc;
+    const int32_t pmin = *std::min_element(p.begin(), p.end()), pmax = *std::max_element(p.begin(), p.end());
+    if (pmin < 0 || pmax >= ROPE_TABLE_MAX_ROWS) {
+        bc->capturable = false;   // served by the per-token table, built while the node is issued
+        return B200_STATUS_SUCCESS;
+    }
+    return rope_reserve(bc, rope_param_key(op, factors), pmax, [&](const std::vector<int32_t> &all) {
+        return rope_fill_host(bc, op, all.data(), (int64_t)all.size(), factors);
+    });
 }
 
 static int compute_rope(BackendCtx *bc, const ggml_tensor *op) {
@@ -879,6 +967,134 @@ static int compute_rope(BackendCtx *bc, const ggml_tensor *op) {
     }
     return b200_rope((const float *)x->data, (int64_t)x->nb[1], (int64_t)x->nb[2], (float *)op->data, (int64_t)op->nb[1],
                      (int64_t)op->nb[2], bc->rope_dev, nullptr, 0, ne0, n_head, n_tok, op->op_params[1], op->op_params[2], bc->stream);
+}
+
+// ---- ops of decoders with dense weights --------------------------------------------------------------------
+// Rotary (cos, sin) pairs of a latent-attention node's positions: angles in double precision, position * base^(-2 i / dims)
+static std::vector<int32_t> latent_rope_key(const ggml_tensor *op) { return {0x4c61744e, op->op_params[8], op->op_params[9]}; }
+static bool latent_rotates(const ggml_tensor *op) {
+    return (op->op == B200_OP_LATENT_STORE || op->op == B200_OP_LATENT_QUERY || op->op == B200_OP_LATENT_ATTN) && op->op_params[9] > 0;
+}
+static int latent_rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
+    const ggml_tensor *pos = op->src[1];
+    std::vector<int32_t> p;
+    if (in_our_buffer(pos)) {
+        BufferCtx *c = bctx(pos->buffer);
+        std::lock_guard<std::mutex> lk(c->mu);
+        auto it = c->i32_shadow.find(pos->data);
+        if (it != c->i32_shadow.end()) p = it->second;
+    }
+    if (p.empty()) {
+        bc->capturable = false;
+        p.resize(pos->ne[0]);
+        B200_CUDA(cudaStreamSynchronize(bc->stream));
+        B200_CUDA(cudaMemcpy(p.data(), pos->data, p.size() * 4, cudaMemcpyDeviceToHost));
+    }
+    const int32_t pmin = *std::min_element(p.begin(), p.end()), pmax = *std::max_element(p.begin(), p.end());
+    B200_REQUIRE(pmin >= 0 && pmax < ROPE_TABLE_MAX_ROWS, "latent attention: position %d out of range", pmin < 0 ? pmin : pmax);
+    const int dims = op->op_params[9];
+    const double base = (double)param_f32(op, 8);
+    return rope_reserve(bc, latent_rope_key(op), pmax, [&](const std::vector<int32_t> &all) {
+        bc->rope_host.resize(all.size() * (size_t)dims);
+        for (int i = 0; i < dims / 2; i++) {
+            const double f = pow(base, -2.0 * i / dims);
+            for (size_t r = 0; r < all.size(); r++) {
+                bc->rope_host[r * dims + 2 * i] = (float)cos((double)all[r] * f);
+                bc->rope_host[r * dims + 2 * i + 1] = (float)sin((double)all[r] * f);
+            }
+        }
+        return (int)B200_STATUS_SUCCESS;
+    });
+}
+
+static int compute_dense_mm(BackendCtx *bc, const ggml_tensor *op) {
+    const ggml_tensor *w = op->src[0], *x = op->src[1], *add = op->src[2], *nw = op->src[3];
+    DenseMm d;
+    d.w = w->data; d.w_type = w->type;
+    d.x = x->data; d.x_type = x->type; d.ldx = row_ld(x);
+    d.y = op->data; d.y_type = op->type; d.ldy = row_ld(op);
+    d.addend = add ? (const float *)add->data : nullptr;
+    d.ld_addend = add ? row_ld(add) : 0;
+    d.norm_w = nw ? (const float *)nw->data : nullptr;
+    d.act = op->op_params[0];
+    d.eps = param_f32(op, 1);
+    d.n = w->ne[1]; d.k = w->ne[0]; d.m = x->ne[1];
+    return launch_dense_mm(d, bc->stream);
+}
+static int compute_gla(BackendCtx *bc, const ggml_tensor *op) {
+    const int32_t *p = op->op_params;
+    GlaArgs a;
+    a.proj = (const float *)op->src[0]->data; a.ldp = row_ld(op->src[0]); a.n = op->src[0]->ne[1];
+    a.a2 = op->src[1]->data; a.a2_type = op->src[1]->type;
+    a.a2_bias = (const float *)op->src[2]->data;
+    a.norm_w = (const float *)op->src[3]->data;
+    a.state = (float *)op->src[4]->data;
+    a.seg = (const int32_t *)op->src[5]->data; a.n_seg = op->src[5]->ne[1];
+    a.scratch = op->src[6] ? (float *)op->src[6]->data : nullptr;
+    a.y = op->data; a.y_type = op->type; a.ldy = row_ld(op);
+    a.heads = p[0]; a.dim = p[1]; a.vdim = p[2]; a.rank = p[12];
+    a.off_q = p[3]; a.off_k = p[4]; a.off_v = p[5]; a.off_g = p[6]; a.off_a = p[7];
+    a.q_factor = param_f32(op, 8); a.inv_tau = param_f32(op, 9); a.eps = param_f32(op, 10);
+    return launch_gla(a, bc->stream);
+}
+static int compute_latent(BackendCtx *bc, const ggml_tensor *op) {
+    const int32_t *p = op->op_params;
+    LatentArgs a;
+    a.heads = p[0]; a.dim = p[1]; a.rot = p[2]; a.rank = p[3]; a.vdim = p[4]; a.window = p[5]; a.rot_dims = p[9];
+    a.scale = param_f32(op, 6); a.eps = param_f32(op, 7);
+    a.off_q = p[10]; a.off_c = p[11]; a.off_g = p[12];
+    a.per_split = p[13]; a.n_splits = p[14];
+    a.pos = (const int32_t *)op->src[1]->data;
+    if (latent_rotates(op)) {
+        const std::vector<int32_t> key = latent_rope_key(op);
+        for (auto &t : bc->rope_by_pos)
+            if (t.key == key && t.dev) { a.rope = t.dev; a.rope_rows = t.rows; }
+        B200_REQUIRE(a.rope != nullptr, "latent attention: no rotary table");
+    }
+    const auto proj = [&](const ggml_tensor *t) { a.proj = (const float *)t->data; a.ldp = row_ld(t); a.n = t->ne[1]; };
+    const auto cells = [&](const ggml_tensor *t) { a.cache = t->data; a.ldc = row_ld(t); a.n_cells = t->ne[1]; a.type = t->type; };
+    const auto result = [&]() { a.y = op->data; a.y_type = op->type; a.ldy = row_ld(op); };
+    switch (op->op) {
+        case B200_OP_LATENT_STORE:
+            proj(op->src[0]);
+            a.norm_w = (const float *)op->src[2]->data;
+            a.cells = (const int32_t *)op->src[3]->data;
+            cells(op);
+            return launch_latent_store(a, bc->stream);
+        case B200_OP_LATENT_QUERY:
+            proj(op->src[0]);
+            a.norm_w = (const float *)op->src[2]->data;
+            a.cells = (const int32_t *)op->src[3]->data;
+            a.ukv = op->src[4]->data;
+            cells(op->src[5]);
+            a.queries = (float *)op->data;
+            return launch_latent_query(a, bc->stream);
+        case B200_OP_LATENT_DECODE:
+            a.queries = (float *)op->src[0]->data;
+            a.n = op->src[0]->ne[2];
+            a.proj = a.queries;
+            cells(op->src[2]);
+            a.row_seg = (const int32_t *)op->src[3]->data;
+            a.seg = (const int32_t *)op->src[4]->data; a.n_seg = op->src[4]->ne[1];
+            a.tab = (const int32_t *)op->src[5]->data; a.n_tab = op->src[5]->ne[0];
+            a.partial = (float *)op->data;
+            return launch_latent_decode(a, bc->stream);
+        case B200_OP_LATENT_VALUE:
+            a.partial = (float *)op->src[0]->data;
+            a.ukv = op->src[2]->data; a.type = op->src[2]->type;
+            proj(op->src[3]);
+            a.sink = (const float *)op->src[4]->data;
+            result();
+            return launch_latent_value(a, bc->stream);
+        default:
+            proj(op->src[0]);
+            a.kv = op->src[2]->data; a.ldkv = row_ld(op->src[2]); a.n_tab = op->src[2]->ne[1];
+            cells(op->src[3]);
+            a.sink = (const float *)op->src[4]->data;
+            a.seg = (const int32_t *)op->src[5]->data; a.n_seg = op->src[5]->ne[1];
+            result();
+            return launch_latent_attn(a, bc->stream);
+    }
 }
 
 static int compute_set_rows(BackendCtx *bc, const ggml_tensor *op) {
@@ -1581,6 +1797,19 @@ static int run_nodes(BackendCtx *bc, ggml_cgraph *g) {
             }
             case GGML_OP_GET_ROWS: rc = compute_get_rows(bc, op); break;
             case GGML_OP_ARGMAX: rc = compute_argmax(bc, op); break;
+            case B200_OP_DENSE_MM: rc = compute_dense_mm(bc, op); break;
+            case B200_OP_RMS_NORM_W:
+                rc = launch_rms_norm_w((const float *)op->src[0]->data, row_ld(op->src[0]), (const float *)op->src[1]->data, op->data, op->type, row_ld(op),
+                                       op->ne[0], op->ne[1], param_f32(op, 0), bc->stream);
+                break;
+            case B200_OP_TAKE_ROWS:
+                rc = launch_take_rows(op->src[0]->data, op->src[0]->type, row_ld(op->src[0]), op->src[0]->ne[1], (const int32_t *)op->src[1]->data, op->ne[1],
+                                      op->data, op->type, row_ld(op), op->ne[0], param_f32(op, 0), bc->stream);
+                break;
+            case B200_OP_GLA: rc = compute_gla(bc, op); break;
+            case B200_OP_LATENT_STORE: case B200_OP_LATENT_QUERY: case B200_OP_LATENT_DECODE: case B200_OP_LATENT_VALUE: case B200_OP_LATENT_ATTN:
+                rc = compute_latent(bc, op);
+                break;
             case B200_OP_TP_ALL_REDUCE:
                 rc = tp_all_reduce(bc->tp, (float *)op->data, (int64_t)(ggml_nbytes(op) / 4), bc->stream, &bc->capturable);
                 break;
@@ -1660,6 +1889,10 @@ static int backend_graph_compute(ggml_backend_t be, ggml_cgraph *g) {
         const ggml_tensor *op = g->nodes[i];
         if (op && op->op == GGML_OP_ROPE && supports_glue(op, nullptr)) {
             int rc = rope_prepare(bc, op);
+            if (rc != B200_STATUS_SUCCESS) return rc;
+        }
+        if (op && latent_rotates(op) && supports_dense(op, nullptr)) {
+            int rc = latent_rope_prepare(bc, op);
             if (rc != B200_STATUS_SUCCESS) return rc;
         }
         if (op && (op->op == B200_OP_TP_ALL_REDUCE || op->op == B200_OP_TP_ALL_GATHER)) {

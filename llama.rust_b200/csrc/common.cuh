@@ -239,6 +239,89 @@ int launch_get_rows(int type, const void *table, int64_t ne0, int64_t table_rows
                     int64_t out_stride, cudaStream_t s);
 int launch_argmax(const float *x, int64_t x_stride, int64_t ne0, int64_t nrows, int32_t *out, cudaStream_t s);
 
+// dense mat-muls (dense_mm.cu): y[m][n] = act(w x') + addend with w [n][k] F32 or BF16 rows, x [m][k] F32 or BF16 rows and, with
+// norm_w, x' = x / rms(x) * norm_w (few rows only)
+constexpr int DENSE_FEW_ROWS = 16;   // activation rows up to which the weights are read row by row
+struct DenseMm {
+    const void *w = nullptr;
+    int w_type = 0;
+    const void *x = nullptr;
+    int x_type = 0;
+    int64_t ldx = 0;                 // elements
+    void *y = nullptr;
+    int y_type = 0;
+    int64_t ldy = 0;
+    const float *addend = nullptr;
+    int64_t ld_addend = 0;
+    const float *norm_w = nullptr;
+    float eps = 0.0f;
+    int act = 0;                     // 0: none, 1: tanh-form gelu
+    int64_t n = 0, k = 0, m = 0;
+};
+int launch_dense_mm(const DenseMm &d, cudaStream_t s);
+bool gemm_bf16_takes(const DenseMm &d);                         // gemm_bf16_tcgen05.cu
+int launch_gemm_bf16(const DenseMm &d, cudaStream_t s);
+// weighted RMS norm of F32 rows into F32 or BF16 rows; rows of a table by index times a factor (dense_mm.cu)
+int launch_rms_norm_w(const float *x, int64_t ldx, const float *w, void *y, int y_type, int64_t ldy, int64_t ne0, int64_t nrows, float eps, cudaStream_t s);
+int launch_take_rows(const void *table, int table_type, int64_t ld_table, int64_t table_rows, const int32_t *ids, int64_t n, void *y, int y_type, int64_t ldy,
+                     int64_t ne0, float factor, cudaStream_t s);
+
+// gated linear attention (gla.cu)
+struct GlaArgs {
+    const float *proj = nullptr;     // [n][ldp]: q, k, v, g and the decay's low-rank input at the offsets
+    int64_t ldp = 0, n = 0;
+    const void *a2 = nullptr;        // [heads dim][rank] F32 or BF16
+    int a2_type = 0;
+    const float *a2_bias = nullptr, *norm_w = nullptr;
+    float *state = nullptr;          // [slot][heads][dim][vdim]
+    const int32_t *seg = nullptr;
+    int64_t n_seg = 0;
+    float *scratch = nullptr;        // null: token by token
+    void *y = nullptr;
+    int y_type = 0;
+    int64_t ldy = 0;
+    int heads = 0, dim = 0, vdim = 0, rank = 0;
+    int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a = 0;
+    float q_factor = 1.0f, inv_tau = 1.0f, eps = 0.0f;
+};
+size_t gla_scratch_floats(int64_t heads, int64_t dim, int64_t vdim, int64_t n, int64_t n_seg);
+int launch_gla(const GlaArgs &a, cudaStream_t s);
+
+// latent attention (latent_attn.cu)
+struct LatentArgs {
+    int heads = 0, dim = 0, rot = 0, rank = 0, vdim = 0, window = 0, rot_dims = 0;
+    float scale = 1.0f, eps = 0.0f;
+    int off_q = 0, off_c = 0, off_g = 0;
+    int per_split = 0, n_splits = 0;
+    int64_t n = 0;
+    const float *proj = nullptr;     // [n][ldp]
+    int64_t ldp = 0;
+    const int32_t *pos = nullptr;
+    const float *norm_w = nullptr;   // [rank]
+    const float *rope = nullptr;     // [rope_rows][rot_dims]: (cos, sin) pairs by position
+    int64_t rope_rows = 0;
+    const int32_t *cells = nullptr;  // the cell each row is stored in
+    const void *ukv = nullptr;       // [heads (dim + vdim)][rank]
+    int type = 0;                    // of ukv, the cell rows and the expanded rows: F32 or BF16
+    void *cache = nullptr;           // [n_cells][ldc]
+    int64_t ldc = 0, n_cells = 0;
+    const int32_t *row_seg = nullptr, *seg = nullptr, *tab = nullptr;
+    int64_t n_seg = 0, n_tab = 0;
+    float *queries = nullptr;        // [n][heads][rank + rot]
+    float *partial = nullptr;        // [n][n_splits][heads][rank + 2]
+    const void *kv = nullptr;        // [n_tab][ldkv]: heads x dim keys, heads x vdim values
+    int64_t ldkv = 0;
+    const float *sink = nullptr;
+    void *y = nullptr;
+    int y_type = 0;
+    int64_t ldy = 0;
+};
+int launch_latent_store(const LatentArgs &a, cudaStream_t s);
+int launch_latent_query(const LatentArgs &a, cudaStream_t s);
+int launch_latent_decode(const LatentArgs &a, cudaStream_t s);
+int launch_latent_value(const LatentArgs &a, cudaStream_t s);
+int launch_latent_attn(const LatentArgs &a, cudaStream_t s);   // cache: the rows by tab entry (ldc apart)
+
 // scratch owned by the library (one growing allocation per device)
 int scratch_get(size_t bytes, void **ptr);
 int scratch_get_kx(size_t bytes, void **ptr);   // a second block, for the K-split exchange of the decode mat-mul
@@ -281,6 +364,26 @@ bool pdl_enabled();
 int numerics_mode();
 void set_numerics_mode(int mode);
 #ifdef __CUDACC__
+// the same with clusters of cluster_x blocks along x
+template <typename... KArgs, typename... Args>
+inline int launch_pdl_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, unsigned cluster_x, size_t smem, cudaStream_t s, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cluster_x;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    B200_CUDA(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
+    return B200_STATUS_SUCCESS;
+}
 template <typename... KArgs, typename... Args>
 inline int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
     cudaLaunchConfig_t cfg = {};

@@ -1,302 +1,21 @@
-// A Llama decode driver over the ggml backend plug-in (include/llama_b200.h).
+// A decode driver over the ggml backend plug-in (include/llama_b200.h).
 //
 // The reference's DecodeContext (crates/llama/src/context.rs) owns the weights, the KV cache and the
 // per-step input tensors, builds the forward graph and hands it to a backend.  This file does the same
-// for the llama architecture with this library's own backend, and it talks to that backend only
+// with this library's own backend, and it talks to that backend only
 // through the vtables a foreign host would use: get_alloc_size / alloc_buffer / set_tensor /
-// graph_compute / get_tensor_async.  The nodes are emitted in the order the reference's graph gets them
-// (depth-first from the roots it expands: each layer's input, the two cache writes, the logits).
-#include <algorithm>
+// graph_compute / get_tensor_async.  The nodes of a step come from the context's architecture (arch_*.cpp).
 #include <cmath>
-#include <cstring>
-#include <deque>
-#include <map>
-#include <memory>
-#include <string>
-#include <vector>
 
-#include "common.cuh"
-#include "ggml_b200_backend.h"
-#include "llama_b200.h"
-#include "tp.h"
+#include "decode_ctx.h"
 
 using namespace b200;
 
 namespace {
 
-constexpr size_t ALIGN = 256;
-constexpr int64_t KV_PAD = 256;   // crates/llama/src/kv_cache.rs:1887-1917: n_kv is padded to 256 cells
-
-size_t type_size(int type) {
-    switch (type) {
-        case B200_TYPE_F32: case B200_TYPE_I32: return 4;
-        case B200_TYPE_F16: return 2;
-        case B200_TYPE_I64: return 8;
-        default: return 0;
-    }
-}
-size_t quant_row_bytes(int type, int64_t ne0) { return (size_t)(ne0 / GROUP_K) * group_src_bytes(type); }
-
-struct Weight {
-    ggml_tensor t;
-    ggml_backend_buffer_t buf = nullptr;
-};
-
-struct Graph {
-    std::deque<ggml_tensor> tensors;      // stable addresses
-    std::vector<ggml_tensor *> nodes;
-    ggml_tensor *tokens = nullptr, *pos = nullptr, *mask = nullptr, *row_idx = nullptr, *out_ids = nullptr;
-    ggml_tensor *logits = nullptr, *argmax = nullptr;
-    size_t bytes = 0;                     // compute-buffer bytes the graph spans
-};
-
-}  // namespace
-
-struct b200_llama {
-    b200_llama_hparams hp;
-    int32_t n_ctx = 0, n_batch = 0;
-    ggml_backend_dev_t dev = nullptr;
-    ggml_backend_t backend = nullptr;
-    ggml_backend_buffer_type_t buft = nullptr;
-    void *stream = nullptr;
-    std::map<std::string, std::unique_ptr<Weight>> weights;
-    ggml_backend_buffer_t kv_buf = nullptr, compute_buf = nullptr;
-    std::vector<ggml_tensor> k_l, v_l;    // [n_embd_k_gqa, n_ctx] F16 per layer
-    std::vector<int32_t> cell_pos;        // position held by each cache cell, -1 = empty
-    std::vector<int32_t> cell_seq;        // the sequence the cell belongs to
-    int32_t used = 0;
-    std::map<std::pair<int64_t, int64_t>, std::unique_ptr<Graph>> graphs;   // by (n_tokens, n_kv)
-    Graph *last = nullptr;
-    std::vector<uint16_t> mask_host;
-    std::vector<int64_t> idx_host;
-    // tensor parallel: this rank holds n_head / tp_size heads, n_head_kv / tp_size cache heads, the matching
-    // rows / columns of every matrix (tp.cpp) and 1 / tp_size of the vocabulary rows
-    int32_t tp_rank = 0, tp_size = 1;
-    TpGroup *tp = nullptr;
-    std::vector<uint8_t> shard_tmp;
-};
-
-namespace {
-
-void init_tensor(ggml_tensor *t, int type, int64_t ne0, int64_t ne1 = 1, int64_t ne2 = 1, int64_t ne3 = 1) {
-    memset(t, 0, sizeof(*t));
-    t->type = type;
-    t->ne[0] = ne0; t->ne[1] = ne1; t->ne[2] = ne2; t->ne[3] = ne3;
-    const size_t row = is_quant_type(type) ? quant_row_bytes(type, ne0) : type_size(type) * (size_t)ne0;
-    t->nb[0] = is_quant_type(type) ? (size_t)group_src_bytes(type) / (type == B200_TYPE_Q4_K || type == B200_TYPE_Q6_K ? 1 : 8) : type_size(type);
-    t->nb[1] = row;
-    t->nb[2] = t->nb[1] * (size_t)ne1;
-    t->nb[3] = t->nb[2] * (size_t)ne2;
-}
-
-// One pass over the compute buffer: tensors are placed back to back; a layer's intermediates are
-// placed again over the previous layer's (everything runs in order on one stream).
-struct Builder {
-    b200_llama *c;
-    Graph *g;
-    uint8_t *base;
-    size_t off = 0, high = 0;
-
-    ggml_tensor *fresh(int type, int64_t ne0, int64_t ne1 = 1, int64_t ne2 = 1, int64_t ne3 = 1) {
-        g->tensors.emplace_back();
-        ggml_tensor *t = &g->tensors.back();
-        init_tensor(t, type, ne0, ne1, ne2, ne3);
-        return t;
-    }
-    ggml_tensor *alloc(int type, int64_t ne0, int64_t ne1 = 1, int64_t ne2 = 1, const char *name = "") {
-        ggml_tensor *t = fresh(type, ne0, ne1, ne2);
-        off = (off + ALIGN - 1) / ALIGN * ALIGN;
-        t->data = base ? base + off : nullptr;
-        t->buffer = c->compute_buf;
-        off += t->nb[3];
-        high = std::max(high, off);
-        snprintf(t->name, sizeof(t->name), "%s", name);
-        return t;
-    }
-    ggml_tensor *op(ggml_tensor *t, int code, ggml_tensor *a, ggml_tensor *b = nullptr, ggml_tensor *c2 = nullptr, ggml_tensor *d = nullptr) {
-        t->op = code;
-        t->src[0] = a; t->src[1] = b; t->src[2] = c2; t->src[3] = d;
-        g->nodes.push_back(t);
-        return t;
-    }
-    // an alias of src's bytes with its own shape and strides (RESHAPE / VIEW / PERMUTE nodes)
-    ggml_tensor *alias(int code, ggml_tensor *src, size_t offset, const int64_t ne[4], const size_t nb[4], const char *name = "") {
-        ggml_tensor *t = fresh(src->type, 1);
-        for (int i = 0; i < 4; i++) { t->ne[i] = ne[i]; t->nb[i] = nb[i]; }
-        t->view_src = src->view_src ? src->view_src : src;
-        t->view_offs = src->view_offs + offset;
-        t->data = src->data ? (uint8_t *)src->data + offset : nullptr;
-        t->buffer = src->buffer;
-        snprintf(t->name, sizeof(t->name), "%s", name);
-        return op(t, code, src);
-    }
-    ggml_tensor *reshape_3d(ggml_tensor *a, int64_t ne0, int64_t ne1, int64_t ne2) {
-        const int64_t ne[4] = {ne0, ne1, ne2, 1};
-        const size_t es = a->nb[0];
-        const size_t nb[4] = {es, es * ne0, es * ne0 * ne1, es * ne0 * ne1 * ne2};
-        return alias(GGML_OP_RESHAPE, a, 0, ne, nb);
-    }
-    ggml_tensor *reshape_2d(ggml_tensor *a, int64_t ne0, int64_t ne1) { return reshape_3d(a, ne0, ne1, 1); }
-    ggml_tensor *view_2d(ggml_tensor *a, int64_t ne0, int64_t ne1, size_t nb1, size_t offset) {
-        const int64_t ne[4] = {ne0, ne1, 1, 1};
-        const size_t nb[4] = {a->nb[0], nb1, nb1 * ne1, nb1 * ne1};
-        return alias(GGML_OP_VIEW, a, offset, ne, nb);
-    }
-    ggml_tensor *view_3d(ggml_tensor *a, int64_t ne0, int64_t ne1, int64_t ne2, size_t nb1, size_t nb2, size_t offset) {
-        const int64_t ne[4] = {ne0, ne1, ne2, 1};
-        const size_t nb[4] = {a->nb[0], nb1, nb2, nb2 * ne2};
-        return alias(GGML_OP_VIEW, a, offset, ne, nb);
-    }
-    // permute(a, 0, 2, 1, 3): swap dims 1 and 2
-    ggml_tensor *permute_0213(ggml_tensor *a) {
-        const int64_t ne[4] = {a->ne[0], a->ne[2], a->ne[1], a->ne[3]};
-        const size_t nb[4] = {a->nb[0], a->nb[2], a->nb[1], a->nb[3]};
-        return alias(GGML_OP_PERMUTE, a, 0, ne, nb);
-    }
-    ggml_tensor *mul_mat(ggml_tensor *w, ggml_tensor *x, const char *name = "") {
-        return op(alloc(B200_TYPE_F32, w->ne[1], x->ne[1], 1, name), GGML_OP_MUL_MAT, w, x);
-    }
-    ggml_tensor *binary(int code, ggml_tensor *a, ggml_tensor *b, const char *name = "") {
-        return op(alloc(B200_TYPE_F32, a->ne[0], a->ne[1], a->ne[2], name), code, a, b);
-    }
-    // a new tensor over the bytes of `slot` (the residual stream alternates between two slots)
-    ggml_tensor *over(const ggml_tensor *slot, const char *name) {
-        ggml_tensor *t = fresh(slot->type, slot->ne[0], slot->ne[1], slot->ne[2]);
-        t->data = slot->data;
-        t->buffer = slot->buffer;
-        snprintf(t->name, sizeof(t->name), "%s", name);
-        return t;
-    }
-    ggml_tensor *rms_norm(ggml_tensor *a, float eps) {
-        ggml_tensor *t = op(alloc(B200_TYPE_F32, a->ne[0], a->ne[1], a->ne[2]), GGML_OP_RMS_NORM, a);
-        memcpy(&t->op_params[0], &eps, 4);
-        return t;
-    }
-    // crates/llama/src/graph_arch.rs:1119-1122 build_norm_rms
-    ggml_tensor *norm(ggml_tensor *a, ggml_tensor *w, float eps, const char *name) { return binary(GGML_OP_MUL, rms_norm(a, eps), w, name); }
-    ggml_tensor *silu(ggml_tensor *a) {
-        ggml_tensor *t = op(alloc(B200_TYPE_F32, a->ne[0], a->ne[1], a->ne[2]), GGML_OP_UNARY, a);
-        t->op_params[0] = GGML_UNARY_OP_SILU;
-        return t;
-    }
-    // crates/ggml/src/ops.rs rope_ext: op_params = [n_past, n_dims, mode, n_ctx, n_ctx_orig, freq_base, freq_scale,
-    // ext_factor, attn_factor, beta_fast, beta_slow, sections[4], n_offs]
-    ggml_tensor *rope(ggml_tensor *a, ggml_tensor *pos, const char *name) {
-        const b200_llama_hparams &hp = c->hp;
-        ggml_tensor *t = op(alloc(B200_TYPE_F32, a->ne[0], a->ne[1], a->ne[2], name), GGML_OP_ROPE, a, pos);
-        const float f[6] = {hp.rope_freq_base, hp.rope_freq_scale, 0.0f, 1.0f, 32.0f, 1.0f};
-        t->op_params[1] = hp.n_embd_head;
-        t->op_params[2] = hp.rope_mode;
-        t->op_params[4] = hp.n_ctx_train;
-        memcpy(&t->op_params[5], f, sizeof(f));
-        return t;
-    }
-    // set_rows(cache, rows, idx): the result aliases the cache tensor
-    ggml_tensor *set_rows(ggml_tensor *cache, ggml_tensor *rows, ggml_tensor *idx) {
-        ggml_tensor *t = fresh(cache->type, 1);
-        for (int i = 0; i < 4; i++) { t->ne[i] = cache->ne[i]; t->nb[i] = cache->nb[i]; }
-        t->view_src = cache;
-        t->data = cache->data;
-        t->buffer = cache->buffer;
-        return op(t, GGML_OP_SET_ROWS, rows, idx);
-    }
-    // the sum of a over the ranks of the tensor-parallel group, in place: the node aliases a
-    ggml_tensor *tp_all_reduce(ggml_tensor *a, const char *name) {
-        ggml_tensor *t = fresh(a->type, a->ne[0], a->ne[1], a->ne[2]);
-        t->data = a->data;
-        t->buffer = a->buffer;
-        t->view_src = a->view_src ? a->view_src : a;
-        t->view_offs = a->view_offs;
-        snprintf(t->name, sizeof(t->name), "%s", name);
-        return op(t, B200_OP_TP_ALL_REDUCE, a);
-    }
-    ggml_tensor *get_rows(ggml_tensor *table, ggml_tensor *ids, const char *name = "") {
-        return op(alloc(B200_TYPE_F32, table->ne[0], ids->ne[0], 1, name), GGML_OP_GET_ROWS, table, ids);
-    }
-};
-
-ggml_tensor *weight(b200_llama *c, const std::string &name) {
-    auto it = c->weights.find(name);
-    return it == c->weights.end() ? nullptr : &it->second->t;
-}
-
-// crates/llama/src/graph_arch.rs:106-248 with attn_kv_cached's flash-attention branch (:1173-1240) and
-// build_ffn_silu_par (:1128-1158).  base == nullptr only measures.
-int build_graph(b200_llama *c, Graph *g, uint8_t *base, int64_t n, int64_t n_kv, int64_t n_out) {
-    const b200_llama_hparams &hp = c->hp;
-    const int64_t E = hp.n_embd, HD = hp.n_embd_head, H = hp.n_head / c->tp_size, HK = hp.n_head_kv / c->tp_size, EK = HK * HD;
-    const bool tp = c->tp_size > 1;
-    Builder b{c, g, base};
-    g->tokens = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_tokens");
-    g->pos = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_pos");
-    g->mask = b.alloc(B200_TYPE_F16, n_kv, n, 1, "kq_mask");
-    g->row_idx = b.alloc(B200_TYPE_I64, n, 1, 1, "kv_idxs");
-    g->out_ids = b.alloc(B200_TYPE_I32, n_out, 1, 1, "inp_out_ids");
-    ggml_tensor *resid[2] = {b.alloc(B200_TYPE_F32, E, n, 1, "resid_a"), b.alloc(B200_TYPE_F32, E, n, 1, "resid_b")};
-
-    ggml_tensor *tok_embd = weight(c, "token_embd.weight");
-    B200_REQUIRE(tok_embd != nullptr, "llama: token_embd.weight has not been set");
-    ggml_tensor *inp = b.op(b.over(resid[0], "inp_embd"), GGML_OP_GET_ROWS, tok_embd, g->tokens);
-    const size_t layer_base = b.off;
-    const float kq_scale = 1.0f / sqrtf((float)HD);
-
-    for (int il = 0; il < hp.n_layer; il++) {
-        b.off = layer_base;
-        const std::string p = "blk." + std::to_string(il) + ".";
-        ggml_tensor *wq = weight(c, p + "attn_q.weight"), *wk = weight(c, p + "attn_k.weight"), *wv = weight(c, p + "attn_v.weight");
-        ggml_tensor *wo = weight(c, p + "attn_output.weight"), *an = weight(c, p + "attn_norm.weight"), *fn = weight(c, p + "ffn_norm.weight");
-        ggml_tensor *wg = weight(c, p + "ffn_gate.weight"), *wu = weight(c, p + "ffn_up.weight"), *wd = weight(c, p + "ffn_down.weight");
-        B200_REQUIRE(wq && wk && wv && wo && an && fn && wg && wu && wd, "llama: layer %d is missing a tensor", il);
-
-        ggml_tensor *cur = b.norm(inp, an, hp.norm_rms_eps, "attn_norm");
-        // root 1: the K cache write
-        ggml_tensor *k = b.reshape_3d(b.mul_mat(wk, cur, "Kcur"), HD, HK, n);
-        k = b.rope(k, g->pos, "Kcur_rope");
-        ggml_tensor *k_rows = b.view_2d(k, EK, n, k->nb[2], 0);
-        b.set_rows(&c->k_l[il], k_rows, g->row_idx);
-        // root 2: the V cache write
-        ggml_tensor *v = b.reshape_3d(b.mul_mat(wv, cur, "Vcur"), HD, HK, n);
-        ggml_tensor *v_rows = b.view_2d(v, EK, n, v->nb[2], 0);
-        b.set_rows(&c->v_l[il], v_rows, g->row_idx);
-        // root 3: the layer output, reached through the attention
-        ggml_tensor *q = b.reshape_3d(b.mul_mat(wq, cur, "Qcur"), HD, H, n);
-        q = b.rope(q, g->pos, "Qcur_rope");
-        ggml_tensor *q_fa = b.permute_0213(q);
-        // KvCache::get_k / get_v: [head, n_head_kv, n_kv] views of the layer's cache, then [head, n_kv, n_head_kv]
-        ggml_tensor *k_fa = b.permute_0213(b.view_3d(&c->k_l[il], HD, HK, n_kv, HD * 2, EK * 2, 0));
-        ggml_tensor *v_fa = b.permute_0213(b.view_3d(&c->v_l[il], HD, HK, n_kv, HD * 2, EK * 2, 0));
-        ggml_tensor *fa = b.op(b.alloc(B200_TYPE_F32, HD, H, n, "kqv_out"), GGML_OP_FLASH_ATTN_EXT, q_fa, k_fa, v_fa, g->mask);
-        memcpy(&fa->op_params[0], &kq_scale, 4);
-        ggml_tensor *attn = b.mul_mat(wo, b.reshape_2d(fa, HD * H, n), "attn_out");
-        if (tp) attn = b.tp_all_reduce(attn, "attn_out_sum");   // attn holds the partial sums over this rank's heads
-        ggml_tensor *ffn_inp = b.binary(GGML_OP_ADD, attn, inp, "ffn_inp");
-        cur = b.norm(ffn_inp, fn, hp.norm_rms_eps, "ffn_norm");
-        ggml_tensor *gate = b.silu(b.mul_mat(wg, cur, "ffn_gate"));
-        ggml_tensor *up = b.mul_mat(wu, cur, "ffn_up");
-        ggml_tensor *down = b.mul_mat(wd, b.binary(GGML_OP_MUL, gate, up, "ffn_gate_par"), "ffn_out");
-        if (tp) down = b.tp_all_reduce(down, "ffn_out_sum");   // down holds the partial sums over this rank's FFN rows
-        inp = b.op(b.over(resid[(il + 1) & 1], "l_out"), GGML_OP_ADD, down, ffn_inp);
-    }
-    b.off = layer_base;
-    ggml_tensor *on = weight(c, "output_norm.weight");
-    ggml_tensor *ow = weight(c, "output.weight");
-    if (!ow) ow = tok_embd;   // tied embeddings
-    B200_REQUIRE(on != nullptr, "llama: output_norm.weight has not been set");
-    ggml_tensor *cur = b.norm(inp, on, hp.norm_rms_eps, "result_norm");
-    cur = b.get_rows(cur, g->out_ids, "result_norm_rows");   // crates/llama/src/graph.rs:308-313 out_rows
-    g->logits = b.mul_mat(ow, cur, "result_output");
-    if (tp && ow != tok_embd) {   // this rank's vocabulary rows: gather the full row on every rank
-        ggml_tensor *staging = b.alloc(B200_TYPE_F32, ow->ne[1] * c->tp_size, n_out, 1, "result_output_staging");
-        g->logits = b.op(b.alloc(B200_TYPE_F32, ow->ne[1] * c->tp_size, n_out, 1, "result_output_all"), B200_OP_TP_ALL_GATHER, g->logits, staging);
-    }
-    g->argmax = b.op(b.alloc(B200_TYPE_I32, n_out, 1, 1, "argmax"), GGML_OP_ARGMAX, g->logits);
-    g->bytes = b.high;
-    return B200_STATUS_SUCCESS;
-}
-
-int64_t n_kv_for(const b200_llama *c, int32_t used) {
+int64_t n_kv_for(const b200_llama *c, int32_t high) {
     // min(size, max(256, pad256(highest used cell + 1))): crates/llama/src/kv_cache.rs:1887-1917
-    const int64_t padded = (used + KV_PAD - 1) / KV_PAD * KV_PAD;
+    const int64_t padded = (high + KV_PAD - 1) / KV_PAD * KV_PAD;
     return std::min<int64_t>(c->n_ctx, std::max<int64_t>(KV_PAD, padded));
 }
 
@@ -344,6 +63,50 @@ int b200_llama_tp_exchange_kind(const b200_llama *c) {
     return c->tp->ll_ready ? 1 : 0;
 }
 
+// the context of an architecture: backend, memory, cells and slots
+static int context_new(std::unique_ptr<Arch> arch, int device, int32_t n_ctx, int32_t n_batch, int32_t n_seq, int32_t cpu_threads, int32_t tp_rank,
+                       int32_t tp_size, const void *id128, b200_tp_hook_fn hook, void *hook_user, const b200_llama_hparams *hp, b200_llama **out) {
+    B200_REQUIRE(n_ctx > 0 && n_ctx % KV_PAD == 0, "llama_new: n_ctx %d must be a positive multiple of 256", n_ctx);
+    B200_REQUIRE(n_batch > 0 && n_batch <= n_ctx, "llama_new: n_batch %d out of (0, n_ctx]", n_batch);
+    B200_REQUIRE(n_seq > 0 && n_seq <= 65536, "llama_new: n_seq %d out of range", n_seq);
+    ggml_backend_reg_t reg = ggml_backend_init();
+    B200_REQUIRE(reg != nullptr && reg->api_version == GGML_BACKEND_API_VERSION, "llama_new: backend registry unavailable");
+    ggml_backend_dev_t dev = reg->iface.get_device(reg, (size_t)device);
+    B200_REQUIRE(dev != nullptr, "llama_new: no usable device %d", device);
+    std::unique_ptr<b200_llama> c(new b200_llama());
+    if (hp) c->hp = *hp;
+    else memset(&c->hp, 0, sizeof(c->hp));
+    c->arch = std::move(arch);
+    c->n_ctx = n_ctx;
+    c->n_batch = n_batch;
+    c->n_seq = n_seq;
+    c->dev = dev;
+    c->tp_rank = tp_rank;
+    c->tp_size = tp_size;
+    const std::string params = "cpu_threads=" + std::to_string(cpu_threads > 0 ? cpu_threads : 8);
+    c->backend = dev->iface.init_backend(dev, params.c_str());
+    if (!c->backend) return B200_STATUS_BACKEND_ERROR;
+    c->buft = dev->iface.get_buffer_type(dev);
+    typedef void *(*get_stream_fn)(ggml_backend_t);
+    get_stream_fn get_stream = (get_stream_fn)reg->iface.get_proc_address(reg, "b200_backend_get_stream");
+    c->stream = get_stream ? get_stream(c->backend) : nullptr;
+    int rc = c->arch->alloc_memory(c.get());
+    if (rc != B200_STATUS_SUCCESS) { b200_llama_free(c.release()); return rc; }
+    c->cell_pos.assign(n_ctx, -1);
+    c->cell_seq.assign(n_ctx, -1);
+    c->slot_seq.assign(n_seq, -1);
+    if (tp_size > 1) {
+        rc = tp_group_create(tp_rank, tp_size, device, id128, hook, hook_user, &c->tp);
+        if (rc != B200_STATUS_SUCCESS) { b200_llama_free(c.release()); return rc; }
+        typedef void (*set_tp_fn)(ggml_backend_t, void *);
+        set_tp_fn set_tp = (set_tp_fn)reg->iface.get_proc_address(reg, "b200_backend_set_tp");
+        if (!set_tp) { b200_llama_free(c.release()); B200_REQUIRE(false, "llama_new: the backend has no tensor-parallel entry"); }
+        set_tp(c->backend, c->tp);
+    }
+    *out = c.release();
+    return B200_STATUS_SUCCESS;
+}
+
 static int llama_new_impl(const b200_llama_hparams *hp, int device, int32_t n_ctx, int32_t n_batch, int32_t cpu_threads, int32_t tp_rank,
                           int32_t tp_size, const void *id128, b200_tp_hook_fn hook, void *hook_user, b200_llama **out) {
     B200_REQUIRE(hp != nullptr && out != nullptr, "llama_new: null argument");
@@ -361,56 +124,39 @@ static int llama_new_impl(const b200_llama_hparams *hp, int device, int32_t n_ct
     B200_REQUIRE(hp->rope_mode == 0 || hp->rope_mode == 2, "llama_new: rope mode %d is neither NORMAL (0) nor NEOX (2)", hp->rope_mode);
     B200_REQUIRE((hp->n_head / tp_size * hp->n_embd_head) % GROUP_K == 0 && (hp->n_ff / tp_size) % GROUP_K == 0 && hp->n_ff % tp_size == 0,
                  "llama_new: a rank's share of the heads and of n_ff must be multiples of 256 elements");
-    B200_REQUIRE(n_ctx > 0 && n_ctx % KV_PAD == 0, "llama_new: n_ctx %d must be a positive multiple of 256", n_ctx);
-    B200_REQUIRE(n_batch > 0 && n_batch <= n_ctx, "llama_new: n_batch %d out of (0, n_ctx]", n_batch);
-    ggml_backend_reg_t reg = ggml_backend_init();
-    B200_REQUIRE(reg != nullptr && reg->api_version == GGML_BACKEND_API_VERSION, "llama_new: backend registry unavailable");
-    ggml_backend_dev_t dev = reg->iface.get_device(reg, (size_t)device);
-    B200_REQUIRE(dev != nullptr, "llama_new: no usable device %d", device);
-    std::unique_ptr<b200_llama> c(new b200_llama());
-    c->hp = *hp;
-    c->n_ctx = n_ctx;
-    c->n_batch = n_batch;
-    c->dev = dev;
-    c->tp_rank = tp_rank;
-    c->tp_size = tp_size;
-    const std::string params = "cpu_threads=" + std::to_string(cpu_threads > 0 ? cpu_threads : 8);
-    c->backend = dev->iface.init_backend(dev, params.c_str());
-    if (!c->backend) return B200_STATUS_BACKEND_ERROR;
-    c->buft = dev->iface.get_buffer_type(dev);
-    typedef void *(*get_stream_fn)(ggml_backend_t);
-    get_stream_fn get_stream = (get_stream_fn)reg->iface.get_proc_address(reg, "b200_backend_get_stream");
-    c->stream = get_stream ? get_stream(c->backend) : nullptr;
+    return context_new(make_llama_arch(*hp), device, n_ctx, n_batch, n_ctx, cpu_threads, tp_rank, tp_size, id128, hook, hook_user, hp, out);
+}
 
-    // KV cache: per layer K and V, [n_embd_k_gqa, n_ctx] F16, zero-filled
-    const int64_t EK = (int64_t)hp->n_head_kv / tp_size * hp->n_embd_head;
-    const size_t per = ((size_t)EK * 2 * n_ctx + ALIGN - 1) / ALIGN * ALIGN;
-    c->kv_buf = c->buft->iface.alloc_buffer(c->buft, per * 2 * hp->n_layer);
-    if (!c->kv_buf) { b200_llama_free(c.release()); return B200_STATUS_ALLOC_FAILED; }
-    c->kv_buf->iface.clear(c->kv_buf, 0);
-    c->k_l.resize(hp->n_layer);
-    c->v_l.resize(hp->n_layer);
-    uint8_t *kvb = (uint8_t *)c->kv_buf->iface.get_base(c->kv_buf);
-    for (int il = 0; il < hp->n_layer; il++) {
-        for (int which = 0; which < 2; which++) {
-            ggml_tensor *t = which ? &c->v_l[il] : &c->k_l[il];
-            init_tensor(t, B200_TYPE_F16, EK, n_ctx);
-            t->buffer = c->kv_buf;
-            t->data = kvb + per * (2 * il + which);
-            snprintf(t->name, sizeof(t->name), "cache_%c_l%d", which ? 'v' : 'k', il);
-        }
+// ---- architectures described by a configuration file -------------------------------------------------------
+static const struct { const char *name; ArchFromConfig from_config; } CONFIG_ARCHS[] = {
+    {"Rukusun", rukusun_from_config},
+};
+
+int b200_model_new(const char *config_json, int dtype, int device, int32_t n_ctx, int32_t n_batch, int32_t n_seq, b200_llama **out) {
+    B200_REQUIRE(config_json != nullptr && out != nullptr, "model_new: null argument");
+    *out = nullptr;
+    B200_REQUIRE(dtype == B200_TYPE_BF16 || dtype == B200_TYPE_F32, "model_new: weights are kept in BF16 or F32, not type %d", dtype);
+    Json config;
+    B200_REQUIRE(Json::parse(config_json, strlen(config_json), &config) && config.kind == Json::OBJ, "model_new: the configuration is not a JSON object");
+    const Json *name = config.find("architecture");
+    B200_REQUIRE(name != nullptr && name->kind == Json::STR, "model_new: the configuration names no architecture");
+    for (const auto &e : CONFIG_ARCHS) {
+        if (name->str != e.name) continue;
+        std::string err;
+        std::unique_ptr<Arch> arch = e.from_config(config, dtype, &err);
+        B200_REQUIRE(arch != nullptr, "model_new: %s", err.c_str());
+        // a context's memory depends on the sizes in the configuration alone
+        return context_new(std::move(arch), device, n_ctx, n_batch, n_seq, 0, 0, 1, nullptr, nullptr, nullptr, nullptr, out);
     }
-    c->cell_pos.assign(n_ctx, -1);
-    c->cell_seq.assign(n_ctx, -1);
-    if (tp_size > 1) {
-        int rc = tp_group_create(tp_rank, tp_size, device, id128, hook, hook_user, &c->tp);
-        if (rc != B200_STATUS_SUCCESS) { b200_llama_free(c.release()); return rc; }
-        typedef void (*set_tp_fn)(ggml_backend_t, void *);
-        set_tp_fn set_tp = (set_tp_fn)reg->iface.get_proc_address(reg, "b200_backend_set_tp");
-        if (!set_tp) { b200_llama_free(c.release()); B200_REQUIRE(false, "llama_new: the backend has no tensor-parallel entry"); }
-        set_tp(c->backend, c->tp);
-    }
-    *out = c.release();
+    B200_REQUIRE(false, "model_new: architecture %s is not one of this library's", name->str.c_str());
+}
+
+int32_t b200_llama_n_vocab(const b200_llama *c) { return c ? c->arch->n_vocab() : 0; }
+const char *b200_llama_arch_name(const b200_llama *c) { return c ? c->arch->name() : ""; }
+int32_t b200_llama_n_tensors(const b200_llama *c) { return c ? (int32_t)c->arch->tensor_names().size() : 0; }
+int b200_llama_learn_shape(b200_llama *c, const char *name, int64_t ne0, int64_t ne1) {
+    B200_REQUIRE(c != nullptr && name != nullptr, "llama_learn_shape: null argument");
+    B200_REQUIRE(c->arch->learn_shape(name, ne0, ne1), "llama_learn_shape: %s [%lld, %lld] contradicts an earlier tensor", name, (long long)ne1, (long long)ne0);
     return B200_STATUS_SUCCESS;
 }
 
@@ -436,9 +182,71 @@ int b200_llama_set_tensor_shard(b200_llama *c, const char *name, int type, int64
     return set_tensor_impl(c, name, type, ne0, ne1, data, nbytes, false);
 }
 
+static float host_f32(int type, const void *data, size_t i) {
+    if (type == B200_TYPE_F32) return ((const float *)data)[i];
+    const uint32_t u = (uint32_t)((const uint16_t *)data)[i] << 16;
+    float f;
+    memcpy(&f, &u, 4);
+    return f;
+}
+static uint16_t host_bf16(float f) {   // round to nearest, ties to even
+    uint32_t u;
+    memcpy(&u, &f, 4);
+    if ((u & 0x7fffffffu) > 0x7f800000u) return (uint16_t)(u >> 16 | 0x40);
+    return (uint16_t)((u + 0x7fffu + (u >> 16 & 1)) >> 16);
+}
+
+// A tensor of an architecture that says where its tensors go: converted to the type the device tensor holds and copied to its rows
+// there (a device tensor may be put together from several of the model's).
+static int set_placed_tensor(b200_llama *c, const char *name, int type, int64_t ne0, int64_t ne1, const void *data, size_t nbytes) {
+    B200_REQUIRE(type == B200_TYPE_F32 || type == B200_TYPE_BF16, "llama_set_tensor: %s: type %d is not F32 or BF16", name, type);
+    B200_REQUIRE(nbytes == plain_type_size(type) * (size_t)ne0 * (size_t)ne1, "llama_set_tensor: %s: %zu bytes do not hold %lld x %lld elements", name,
+                 nbytes, (long long)ne1, (long long)ne0);
+    int rc = b200_llama_learn_shape(c, name, ne0, ne1);
+    if (rc != B200_STATUS_SUCCESS) return rc;
+    TensorPlace p;
+    B200_REQUIRE(c->arch->place(name, &p), "llama_set_tensor: %s has no tensor %s", c->arch->name(), name);
+    B200_REQUIRE(p.ne1 > 0, "llama_set_tensor: %s is part of a matrix whose size another tensor tells; set that one first", name);
+    B200_REQUIRE(ne0 == p.ne0 && ne1 == p.rows, "llama_set_tensor: %s is [%lld, %lld], the configuration asks for [%lld, %lld]", name, (long long)ne1,
+                 (long long)ne0, (long long)p.rows, (long long)p.ne0);
+    auto it = c->weights.find(p.dst);
+    if (it == c->weights.end()) {
+        std::unique_ptr<Weight> w(new Weight());
+        init_tensor(&w->t, p.type, p.ne0, p.ne1);
+        snprintf(w->t.name, sizeof(w->t.name), "%s", p.dst.c_str());
+        w->buf = c->buft->iface.alloc_buffer(c->buft, w->t.nb[2] + TENSOR_ALIGN);
+        if (!w->buf) return B200_STATUS_ALLOC_FAILED;
+        w->buf->usage = GGML_BACKEND_BUFFER_USAGE_WEIGHTS;
+        w->t.buffer = w->buf;
+        w->t.data = w->buf->iface.get_base(w->buf);
+        it = c->weights.emplace(p.dst, std::move(w)).first;
+    }
+    ggml_tensor *t = &it->second->t;
+    const size_t count = (size_t)ne0 * (size_t)ne1, offset = (size_t)p.row0 * t->nb[1];
+    std::vector<float> f;
+    std::vector<uint16_t> h;
+    const void *src = data;
+    if (p.type == B200_TYPE_F32 && (type != B200_TYPE_F32 || p.plus_one)) {
+        f.resize(count);
+        for (size_t i = 0; i < count; i++) f[i] = host_f32(type, data, i) + (p.plus_one ? 1.0f : 0.0f);
+        src = f.data();
+    } else if (p.type == B200_TYPE_BF16 && type != B200_TYPE_BF16) {
+        h.resize(count);
+        for (size_t i = 0; i < count; i++) h[i] = host_bf16(((const float *)data)[i]);
+        src = h.data();
+    }
+    c->backend->iface.synchronize(c->backend);
+    t->buffer->iface.set_tensor(t->buffer, t, src, offset, count * plain_type_size(p.type));
+    c->tensors_set.insert(name);
+    c->graphs.clear();
+    c->last = nullptr;
+    return B200_STATUS_SUCCESS;
+}
+
 static int set_tensor_impl(b200_llama *c, const char *name, int type, int64_t ne0, int64_t ne1, const void *data, size_t nbytes, bool whole) {
     B200_REQUIRE(c != nullptr && name != nullptr && data != nullptr, "llama_set_tensor: null argument");
     B200_REQUIRE(ne0 > 0 && ne1 > 0, "llama_set_tensor: %s has an empty shape", name);
+    if (!c->arch->masked_cache()) return set_placed_tensor(c, name, type, ne0, ne1, data, nbytes);
     const bool quant = is_quant_type(type);
     B200_REQUIRE(quant || type == B200_TYPE_F32 || type == B200_TYPE_F16, "llama_set_tensor: %s: type %d is not supported", name, type);
     B200_REQUIRE(!quant || ne0 % GROUP_K == 0, "llama_set_tensor: %s: row length %lld is not a multiple of 256", name, (long long)ne0);
@@ -484,7 +292,28 @@ int b200_llama_kv_clear(b200_llama *c) {
     c->kv_buf->iface.clear(c->kv_buf, 0);
     std::fill(c->cell_pos.begin(), c->cell_pos.end(), -1);
     std::fill(c->cell_seq.begin(), c->cell_seq.end(), -1);
-    c->used = 0;
+    std::fill(c->slot_seq.begin(), c->slot_seq.end(), -1);
+    c->seqs.clear();
+    c->used = c->high = c->first_free = 0;
+    return B200_STATUS_SUCCESS;
+}
+
+static void free_cell(b200_llama *c, int32_t cell) {
+    c->cell_pos[cell] = c->cell_seq[cell] = -1;
+    c->used--;
+    c->first_free = std::min(c->first_free, cell);
+    while (c->high > 0 && c->cell_seq[c->high - 1] < 0) c->high--;
+}
+
+int b200_llama_seq_rm(b200_llama *c, int32_t seq) {
+    B200_REQUIRE(c != nullptr && seq >= 0, "llama_seq_rm: bad argument");
+    for (int32_t j = c->high - 1; j >= 0; j--)
+        if (c->cell_seq[j] == seq) free_cell(c, j);
+    auto it = c->seqs.find(seq);
+    if (it != c->seqs.end()) {
+        if (it->second.slot >= 0) c->slot_seq[it->second.slot] = -1;
+        c->seqs.erase(it);
+    }
     return B200_STATUS_SUCCESS;
 }
 
@@ -492,6 +321,7 @@ int32_t b200_llama_kv_used(const b200_llama *c) { return c ? c->used : 0; }
 
 int b200_llama_get_hparams(const b200_llama *c, b200_llama_hparams *out) {
     B200_REQUIRE(c != nullptr && out != nullptr, "llama_get_hparams: null argument");
+    B200_REQUIRE(c->arch->masked_cache(), "llama_get_hparams: %s is described by its configuration", c->arch->name());
     *out = c->hp;
     return B200_STATUS_SUCCESS;
 }
@@ -502,68 +332,192 @@ int b200_llama_decode(b200_llama *c, const int32_t *tokens, const int32_t *pos, 
     return b200_llama_decode_seqs(c, tokens, pos, nullptr, n, &last, 1, logits, argmax);
 }
 
+// A step of a segmented architecture, on the host: the sequences among its rows, checked (a sequence's rows stand together and
+// continue it), then their cells and slots, and the inputs the nodes read.  Nothing changes before every check has passed.
+static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_ids, int32_t n, StepShape *s) {
+    struct Seg { int32_t seq, row0, rows; int64_t pos0; };
+    std::vector<Seg> segs;
+    for (int32_t i = 0; i < n; i++) {
+        const int32_t q = seq_ids ? seq_ids[i] : 0;
+        B200_REQUIRE(q >= 0, "llama_decode: sequence id %d", q);
+        if (!segs.empty() && segs.back().seq == q) {
+            B200_REQUIRE(pos[i] == pos[i - 1] + 1, "llama_decode: position %d of sequence %d follows %d", pos[i], q, pos[i - 1]);
+            segs.back().rows++;
+            continue;
+        }
+        for (const Seg &o : segs) B200_REQUIRE(o.seq != q, "llama_decode: the rows of sequence %d do not stand together", q);
+        const auto it = c->seqs.find(q);
+        const int64_t want = it == c->seqs.end() ? 0 : it->second.next_pos;
+        B200_REQUIRE(pos[i] == want, "llama_decode: sequence %d continues at position %lld, not %d", q, (long long)want, pos[i]);
+        segs.push_back({q, i, 1, pos[i]});
+    }
+    const int64_t span = c->arch->key_span();
+    int64_t fresh = 0, free_slots = 0;
+    for (const Seg &g : segs) fresh += c->seqs.find(g.seq) == c->seqs.end();
+    for (int32_t q : c->slot_seq) free_slots += q < 0;
+    B200_REQUIRE(fresh <= free_slots, "llama_decode: %lld new sequences, %lld of %d state slots free", (long long)fresh, (long long)free_slots, c->n_seq);
+    B200_REQUIRE(span < 0 || c->used + n <= c->n_ctx, "llama_decode: kv cache full (%d used + %d > %d)", c->used, n, c->n_ctx);
+
+    c->seg_host.assign(segs.size() * SEG_FIELDS, 0);
+    c->row_seg_host.assign(n, 0);
+    c->cells_host.assign(n, 0);
+    c->tab_host.clear();
+    int64_t max_keys = 1, max_rows = 1;
+    for (size_t k = 0; k < segs.size(); k++) {
+        const Seg &g = segs[k];
+        Sequence &q = c->seqs[g.seq];
+        const bool is_new = q.slot < 0;
+        if (is_new) {
+            q.slot = (int32_t)(std::find(c->slot_seq.begin(), c->slot_seq.end(), -1) - c->slot_seq.begin());
+            c->slot_seq[q.slot] = g.seq;
+        }
+        int32_t *f = &c->seg_host[k * SEG_FIELDS];
+        f[SEG_ROW0] = g.row0;
+        f[SEG_ROWS] = g.rows;
+        f[SEG_SLOT] = q.slot;
+        f[SEG_FRESH] = is_new;
+        f[SEG_POS0] = (int32_t)g.pos0;
+        for (int32_t i = 0; i < g.rows; i++) {
+            c->row_seg_host[g.row0 + i] = (int32_t)k;
+            if (span < 0) continue;
+            int32_t cell = c->first_free;
+            while (c->cell_seq[cell] >= 0) cell++;
+            c->first_free = cell + 1;
+            c->cell_pos[cell] = (int32_t)(g.pos0 + i);
+            c->cell_seq[cell] = g.seq;
+            c->used++;
+            c->high = std::max(c->high, cell + 1);
+            c->cells_host[g.row0 + i] = cell;
+            q.cells.push_back(cell);
+        }
+        q.next_pos = g.pos0 + g.rows;
+        max_rows = std::max<int64_t>(max_rows, g.rows);
+        if (span >= 0) {
+            // the positions the first row can see, up to the last row's own
+            const int64_t key0 = span > 0 ? std::max<int64_t>(0, g.pos0 - span + 1) : 0;
+            f[SEG_TAB0] = (int32_t)c->tab_host.size();
+            f[SEG_KEY0] = (int32_t)key0;
+            for (int64_t p = key0; p < q.next_pos; p++) c->tab_host.push_back(q.cells[p - q.kept]);
+            max_keys = std::max(max_keys, q.next_pos - key0);
+        }
+    }
+    s->n_seg = (int64_t)segs.size();
+    s->max_rows = 1;
+    while (s->max_rows < max_rows) s->max_rows *= 2;
+    if (span >= 0) {
+        s->n_tab = std::min<int64_t>(((int64_t)c->tab_host.size() + KV_PAD - 1) / KV_PAD * KV_PAD, (c->n_ctx + KV_PAD - 1) / KV_PAD * KV_PAD);
+        if (max_rows == 1 && span > 0) max_keys = std::min(max_keys, span);
+        s->max_keys = std::min<int64_t>((max_keys + KV_PAD - 1) / KV_PAD * KV_PAD, s->n_tab);
+        c->tab_host.resize(s->n_tab, 0);
+    }
+    return B200_STATUS_SUCCESS;
+}
+// After a step: cells no later token of the sequence can see are free again.
+static void trim_sequences(b200_llama *c, const int32_t *seq_ids, int32_t n) {
+    const int64_t span = c->arch->key_span();
+    if (span <= 0) return;
+    for (int32_t i = 0; i < n; i++) {
+        if (i > 0 && (!seq_ids || seq_ids[i] == seq_ids[i - 1])) continue;
+        Sequence &q = c->seqs[seq_ids ? seq_ids[i] : 0];
+        const int64_t first = std::max<int64_t>(q.kept, q.next_pos - span + 1);
+        for (int64_t p = q.kept; p < first; p++) free_cell(c, q.cells[p - q.kept]);
+        q.cells.erase(q.cells.begin(), q.cells.begin() + (first - q.kept));
+        q.kept = first;
+    }
+}
+
 int b200_llama_decode_seqs(b200_llama *c, const int32_t *tokens, const int32_t *pos, const int32_t *seq_ids, int32_t n,
                            const int32_t *out_rows, int32_t n_out, float *logits, int32_t *argmax) {
     B200_REQUIRE(c != nullptr && tokens != nullptr && pos != nullptr && out_rows != nullptr, "llama_decode: null argument");
     B200_REQUIRE(n > 0 && n <= c->n_batch, "llama_decode: batch size %d out of (0, %d]", n, c->n_batch);
     B200_REQUIRE(n_out > 0 && n_out <= n, "llama_decode: %d output rows for %d tokens", n_out, n);
-    B200_REQUIRE(c->used + n <= c->n_ctx, "llama_decode: kv cache full (%d used + %d > %d)", c->used, n, c->n_ctx);
     for (int i = 0; i < n; i++)
-        B200_REQUIRE(tokens[i] >= 0 && tokens[i] < c->hp.n_vocab, "llama_decode: token %d out of range", tokens[i]);
+        B200_REQUIRE(tokens[i] >= 0 && tokens[i] < c->arch->n_vocab(), "llama_decode: token %d out of range", tokens[i]);
     for (int i = 0; i < n_out; i++) B200_REQUIRE(out_rows[i] >= 0 && out_rows[i] < n, "llama_decode: output row %d out of range", out_rows[i]);
+    const bool masked = c->arch->masked_cache();
 
-    // find_slot + assign: the next free cells, in order; a cell remembers its sequence and position
-    const int32_t head = c->used;
-    const int64_t n_kv = n_kv_for(c, head + n);
+    StepShape shape;
+    shape.n = n;
+    shape.n_out = n_out;
+    if (masked) {
+        B200_REQUIRE(c->used + n <= c->n_ctx, "llama_decode: kv cache full (%d used + %d > %d)", c->used, n, c->n_ctx);
+        // find_slot + assign: the lowest free cells, in order; a cell remembers its sequence and position
+        c->idx_host.resize(n);
+        int32_t cell = c->first_free, high = c->high;
+        for (int i = 0; i < n; i++, cell++) {
+            while (c->cell_seq[cell] >= 0) cell++;
+            c->idx_host[i] = cell;
+            high = std::max(high, cell + 1);
+        }
+        shape.n_kv = n_kv_for(c, high);
+    } else {
+        int rc = plan_segments(c, pos, seq_ids, n, &shape);
+        if (rc != B200_STATUS_SUCCESS) return rc;
+    }
 
-    // the graph for this (n, n_kv, n_out), sized and built once
-    auto key = std::make_pair((int64_t)n * 65536 + n_out, n_kv);
-    auto it = c->graphs.find(key);
+    // the graph for this shape, sized and built once
+    auto it = c->graphs.find(shape);
     if (it == c->graphs.end()) {
         if (!c->compute_buf) {
-            Graph measure;
-            int rc = build_graph(c, &measure, nullptr, c->n_batch, c->n_ctx, c->n_batch);
-            if (rc != B200_STATUS_SUCCESS) return rc;
-            c->compute_buf = c->buft->iface.alloc_buffer(c->buft, measure.bytes + ALIGN);
+            size_t bytes = 0;
+            for (const StepShape &s : c->arch->largest(c)) {
+                Graph measure;
+                int rc = c->arch->build(c, &measure, nullptr, s);
+                if (rc != B200_STATUS_SUCCESS) return rc;
+                bytes = std::max(bytes, measure.bytes);
+            }
+            c->compute_buf = c->buft->iface.alloc_buffer(c->buft, bytes + TENSOR_ALIGN);
             if (!c->compute_buf) return B200_STATUS_ALLOC_FAILED;
             c->compute_buf->usage = GGML_BACKEND_BUFFER_USAGE_COMPUTE;
         }
         std::unique_ptr<Graph> g(new Graph());
-        int rc = build_graph(c, g.get(), (uint8_t *)c->compute_buf->iface.get_base(c->compute_buf), n, n_kv, n_out);
+        int rc = c->arch->build(c, g.get(), (uint8_t *)c->compute_buf->iface.get_base(c->compute_buf), shape);
         if (rc != B200_STATUS_SUCCESS) return rc;
         B200_REQUIRE(g->bytes <= c->compute_buf->size, "llama_decode: graph needs %zu bytes, compute buffer has %zu", g->bytes, c->compute_buf->size);
-        it = c->graphs.emplace(key, std::move(g)).first;
+        it = c->graphs.emplace(shape, std::move(g)).first;
     }
     Graph *g = it->second.get();
 
-    for (int i = 0; i < n; i++) {
-        c->cell_pos[head + i] = pos[i];
-        c->cell_seq[head + i] = seq_ids ? seq_ids[i] : 0;
+    if (masked) {
+        for (int i = 0; i < n; i++) {
+            const int32_t cell = (int32_t)c->idx_host[i];
+            c->cell_pos[cell] = pos[i];
+            c->cell_seq[cell] = seq_ids ? seq_ids[i] : 0;
+            c->high = std::max(c->high, cell + 1);
+        }
+        c->used += n;
+        c->first_free = (int32_t)c->idx_host[n - 1] + 1;
+        // crates/llama/src/graph.rs:704-724 fill_kq_mask_f16 with the sequence test of llama-kv-cache's set_input_kq_mask:
+        // 0 where the cell belongs to the query's sequence and holds a position <= the query's, -inf elsewhere
+        const int64_t n_kv = shape.n_kv;
+        c->mask_host.assign((size_t)n * n_kv, 0xFC00);
+        for (int i = 0; i < n; i++) {
+            const int32_t s = seq_ids ? seq_ids[i] : 0;
+            for (int64_t j = 0; j < c->high; j++)
+                if (c->cell_seq[j] == s && c->cell_pos[j] >= 0 && c->cell_pos[j] <= pos[i]) c->mask_host[(size_t)i * n_kv + j] = 0;
+        }
     }
-    c->used = head + n;
-    // crates/llama/src/graph.rs:704-724 fill_kq_mask_f16 with the sequence test of llama-kv-cache's set_input_kq_mask:
-    // 0 where the cell belongs to the query's sequence and holds a position <= the query's, -inf elsewhere
-    c->mask_host.assign((size_t)n * n_kv, 0xFC00);
-    for (int i = 0; i < n; i++) {
-        const int32_t s = seq_ids ? seq_ids[i] : 0;
-        for (int64_t j = 0; j < c->used; j++)
-            if (c->cell_seq[j] == s && c->cell_pos[j] >= 0 && c->cell_pos[j] <= pos[i]) c->mask_host[(size_t)i * n_kv + j] = 0;
-    }
-    c->idx_host.resize(n);
-    for (int i = 0; i < n; i++) c->idx_host[i] = head + i;
 
     // inputs land with synchronous copies after the previous step has drained
     c->backend->iface.synchronize(c->backend);
     set_input_async(c->backend, g->tokens, tokens, (size_t)n * 4);
     set_input_async(c->backend, g->pos, pos, (size_t)n * 4);
-    set_input_async(c->backend, g->mask, c->mask_host.data(), c->mask_host.size() * 2);
-    set_input_async(c->backend, g->row_idx, c->idx_host.data(), (size_t)n * 8);
+    if (masked) {
+        set_input_async(c->backend, g->mask, c->mask_host.data(), c->mask_host.size() * 2);
+        set_input_async(c->backend, g->row_idx, c->idx_host.data(), (size_t)n * 8);
+    } else {
+        set_input_async(c->backend, g->cells, c->cells_host.data(), (size_t)n * 4);
+        set_input_async(c->backend, g->row_seg, c->row_seg_host.data(), (size_t)n * 4);
+        set_input_async(c->backend, g->seg, c->seg_host.data(), c->seg_host.size() * 4);
+        if (!c->tab_host.empty()) set_input_async(c->backend, g->tab, c->tab_host.data(), c->tab_host.size() * 4);
+    }
     set_input_async(c->backend, g->out_ids, out_rows, (size_t)n_out * 4);
 
     int rc = run_graph(c, g, (int)g->nodes.size() - (argmax ? 0 : 1));   // the ARGMAX node is last
     if (rc != B200_STATUS_SUCCESS) return rc;
     c->last = g;
-    if (logits) c->backend->iface.get_tensor_async(c->backend, g->logits, logits, 0, (size_t)c->hp.n_vocab * n_out * 4);
+    if (!masked) trim_sequences(c, seq_ids, n);
+    if (logits) c->backend->iface.get_tensor_async(c->backend, g->logits, logits, 0, (size_t)c->arch->n_vocab() * n_out * 4);
     if (argmax) c->backend->iface.get_tensor_async(c->backend, g->argmax, argmax, 0, (size_t)n_out * 4);
     c->backend->iface.synchronize(c->backend);
     int code = 0;
