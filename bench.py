@@ -1028,9 +1028,160 @@ def case_llama(args):
     gpu.close()
 
 
+# Layers the size of a real model's, by width: the design's two kinds in the proportion 3 : 1, and the llama model of the
+# same width and the same number of weights per layer (its FFN size makes up the difference)
+RUKUSUN_VOCAB = 32000
+
+
+def rukusun_config(width, layers, window=1024):
+    gla = {"type": "gla", "mixer": {"heads": width // 256, "dim": 128, "vdim": 256, "tau": 16.0}, "mlp": {"kind": "dense", "ff": 4 * width}}
+    lat = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": 4 * width},
+           "mixer": {"heads": width // 128, "dim": 128, "rot_dim": 64, "kv_rank": 512, "vdim": 128, "mask": {"size": window}, "scale": 192 ** -0.5,
+                     "rot": {"base": 10000.0, "dims": 64}}}
+    return {"architecture": "Rukusun", "embedding": {"scale": float(width) ** 0.5}, "layers": [lat if i % 4 == 3 else gla for i in range(layers)],
+            "norm": {"eps": 1e-5}, "vocab": RUKUSUN_VOCAB, "width": width}
+
+
+def rukusun_tensors(cfg, rank=16):
+    """(name, BF16 bits) of every tensor: seeded normals of the right spread, large matrices repeat a block of rows"""
+    rng = np.random.default_rng(0)
+    base = rng.standard_normal(1 << 20).astype(np.float32)
+    E, V = cfg["width"], cfg["vocab"]
+
+    def mat(n, k, gain=1.0, mean=0.0):
+        block = (base * (gain / np.sqrt(k)) + mean).astype(np.float32).view(np.uint32)
+        return np.resize(((block + 0x8000) >> 16).astype(np.uint16), (n, k))
+
+    def vec(n, mean, dev):
+        return mat(1, n, dev * np.sqrt(n), mean).reshape(n)
+
+    yield "embed", mat(V, E)
+    yield "head", mat(V, E)
+    yield "final.norm", vec(E, 0.0, 0.1)
+    for i, lay in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", lay["mixer"]
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        yield p + "norm1", vec(E, 0.0, 0.1)
+        yield p + "norm2", vec(E, 0.0, 0.1)
+        yield p + "mlp.up", mat(lay["mlp"]["ff"], E)
+        yield p + "mlp.down", mat(E, lay["mlp"]["ff"])
+        yield p + "mix.o", mat(E, H * e)
+        if lay["type"] == "gla":
+            yield p + "mix.a1", mat(rank, E)
+            yield p + "mix.a2", mat(H * d, rank)
+            yield p + "mix.a2.b", vec(H * d, 2.0, 1.0)
+            yield p + "mix.norm", vec(e, 1.0, 0.1)
+            for n, rows in (("q", H * d), ("k", H * d), ("v", H * e), ("g", H * e)):
+                yield p + "mix." + n, mat(rows, E)
+        else:
+            R, rot = m["kv_rank"], m["rot_dim"]
+            yield p + "mix.q", mat(H * (d + rot), E)
+            yield p + "mix.dkv", mat(R + rot, E)
+            yield p + "mix.dkv.norm", vec(R, 1.0, 0.1)
+            yield p + "mix.uk", mat(H * d, R)
+            yield p + "mix.uv", mat(H * e, R)
+            yield p + "mix.sink", vec(H, 0.0, 1.0)
+            yield p + "mix.g", mat(H, E)
+
+
+def build_rukusun(width, layers, n_ctx, n_batch, n_seq=16):
+    load_pkg()
+    ll = importlib.import_module("llama_rust_b200.llama")
+    cfg = rukusun_config(width, layers)
+    gpu = ll.Model(cfg, n_ctx, n_batch, n_seq=n_seq)
+    weights = 0
+    for name, t in rukusun_tensors(cfg):
+        gpu.set_tensors({name: t})
+        if ".mix.norm" not in name and name != "embed":
+            weights += t.size
+    return gpu, cfg, weights
+
+
+def build_equal_llama(width, layers, weights_per_layer, n_ctx, n_batch):
+    load_pkg()
+    sh = load_standalone("shapes")
+    ll = importlib.import_module("llama_rust_b200.llama")
+    syn = load_standalone("synth")
+    attn = 2 * width * width + 2 * width * 1024
+    ff = max(256, round((weights_per_layer - attn) / (3 * width) / 256) * 256)
+    hp = dict(sh.LLAMA3_8B, n_vocab=RUKUSUN_VOCAB, n_embd=width, n_head=width // 128, n_head_kv=8, n_ff=ff, n_layer=layers)
+    gpu = ll.Llama(hp, n_ctx, n_batch)
+    for name, ty, arr, ne0, ne1 in syn.llama_tensors(hp, lambda n: sh.q4_k_m_type(n, layers), tensor_shapes=sh.tensor_shapes):
+        gpu.set_tensor(name, ty, arr, ne0, ne1)
+    return gpu, hp, llama_weight_bytes(ll, hp)
+
+
+def time_model(gpu, vocab, prompt, steps):
+    """prefill of `prompt` tokens and single-token steps after it: (ms, ms device-only) each; the second pass counts"""
+    rng = np.random.default_rng(0)
+    toks = rng.integers(0, vocab, prompt).astype(np.int32)
+    out = None
+    for _ in range(3):
+        gpu.kv_clear()
+        t0 = time.perf_counter()
+        tok = gpu.decode(toks, np.arange(prompt), logits=False, argmax=True)
+        pp = (time.perf_counter() - t0) * 1e3
+        pp_dev = gpu.replay(3) / 3
+        gpu.kv_clear()
+        tok = gpu.decode(toks, np.arange(prompt), logits=False, argmax=True)
+        t0 = time.perf_counter()
+        for i in range(steps):
+            tok = gpu.decode([tok], [prompt + i], logits=False, argmax=True)
+        tg = (time.perf_counter() - t0) * 1e3 / steps
+        out = (pp, pp_dev, tg, gpu.replay(steps) / steps)
+    return out
+
+
+def case_rukusun(args):
+    """`--case rukusun`: prefill and decode throughput of the design at a few widths, beside a llama model of equal size (Q4_K_M,
+    fast numerics).  `rukusun_pp` / `rukusun_tg`: one prompt / R single-token steps of a small model, eager launches."""
+    small = args.case != "rukusun"
+    if small:
+        os.environ["B200_CUDA_GRAPHS"] = "0"
+    b = load_pkg()
+    b.set_device(0)
+    prompt = args.prompt if args.prompt > 16 else 2048
+    if small:
+        gpu, cfg, _ = build_rukusun(args.width, args.layers if args.layers < 32 else 4, 2 * prompt, prompt)
+        toks = np.random.default_rng(0).integers(0, cfg["vocab"], prompt).astype(np.int32)
+        tok = gpu.decode(toks, np.arange(prompt), logits=False, argmax=True)
+        if args.case == "rukusun_tg":
+            for i in range(args.launches):
+                tok = gpu.decode([tok], [prompt + i], logits=False, argmax=True)
+        print(json.dumps({"case": args.case, "width": args.width, "kernel_error": b.kernel_error()}), flush=True)
+        gpu.close()
+        return
+    layers, steps = args.layers if args.layers < 32 else 8, 64
+    hbm, tensor = peak_hbm()[0], peak_tensor()[0]
+    rows = []
+    for width in (1024, 2048, 4096):
+        mon = ClockSampler(0)
+        gpu, cfg, weights = build_rukusun(width, layers, 4096, prompt)
+        mon.start()
+        pp, pp_dev, tg, tg_dev = time_model(gpu, cfg["vocab"], prompt, steps)
+        clocks = mon.stop()
+        gpu.close()
+        head = cfg["vocab"] * width
+        lgpu, hp, lbytes = build_equal_llama(width, layers, (weights - head) / layers, 4096, prompt)
+        lpp, lpp_dev, ltg, ltg_dev = time_model(lgpu, hp["n_vocab"], prompt, steps)
+        lgpu.close()
+        lweights = hp["n_layer"] * (2 * width * width + 2 * width * 1024 + 3 * width * hp["n_ff"])
+        rows.append({
+            "width": width, "layers": layers, "prompt": prompt, "weights_m": round(weights / 1e6), "clocks": clocks,
+            "rukusun": {"prefill_tok_s": prompt / pp_dev * 1e3, "prefill_e2e_tok_s": prompt / pp * 1e3, "decode_tok_s": 1e3 / tg_dev, "decode_e2e_tok_s": 1e3 / tg,
+                        "prefill_of_tensor_peak": 2.0 * (weights - head) * prompt / pp_dev / 1e9 / tensor, "decode_of_hbm_peak": 2.0 * weights / tg_dev / 1e6 / hbm},
+            "llama_q4_k_m": {"n_ff": hp["n_ff"], "weights_m": round((lweights + head) / 1e6), "prefill_tok_s": prompt / lpp_dev * 1e3, "prefill_e2e_tok_s": prompt / lpp * 1e3,
+                             "decode_tok_s": 1e3 / ltg_dev, "decode_e2e_tok_s": 1e3 / ltg,
+                             "prefill_of_tensor_peak": 2.0 * lweights * prompt / lpp_dev / 1e9 / tensor, "decode_of_hbm_peak": lbytes / ltg_dev / 1e6 / hbm}})
+        note(json.dumps(rows[-1]))
+    print(json.dumps({"case": "rukusun", "data": "synthetic", "dtype": "bf16 weights, F32 residual", "sizes": rows, "kernel_error": b.kernel_error()}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "fa", "llama_tg", "llama_pp", "llama_b16"], help="one small case for a profiler")
+    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "fa", "llama_tg", "llama_pp", "llama_b16", "rukusun", "rukusun_pp", "rukusun_tg"],
+                    help="one small case for a profiler; rukusun: that design's throughput beside a llama model of equal size")
+    ap.add_argument("--width", type=int, default=4096, help="--case rukusun_pp / rukusun_tg: model width")
     ap.add_argument("--only", default="4096x4096", help="--case gemv / gemm: the shape NxK")
     ap.add_argument("--cols", type=int, default=512, help="--case gemm: activation rows")
     ap.add_argument("--wtype", default="Q4_K", choices=["Q4_K", "Q6_K"], help="--case gemm: weight type")
@@ -1056,6 +1207,8 @@ def main():
         return case_fa(args)
     if args.case == "gemm":
         return case_gemm(args)
+    if args.case and args.case.startswith("rukusun"):
+        return case_rukusun(args)
     if args.case:
         return case_llama(args)
     rank, world, barrier, reduce_max = dist_setup(args.gpus)

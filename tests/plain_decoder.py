@@ -72,8 +72,8 @@ def gla_recurrence(q, k, v, alpha, state):
     return out, S
 
 
-def gla_mixer(h, w, p, mix, eps, state=None):
-    """h [T, width] -> [T, width] and the state"""
+def gla_mixer(h, w, p, mix, eps, state=None, rnd=lambda x: x):
+    """h [T, width] -> [T, width] and the state; rnd: see Plain"""
     H, d, e, T = mix["heads"], mix["dim"], mix["vdim"], h.shape[0]
     q = (h @ w[p + "q"].T).reshape(T, H, d) * d ** -0.5
     k = (h @ w[p + "k"].T).reshape(T, H, d)
@@ -83,7 +83,7 @@ def gla_mixer(h, w, p, mix, eps, state=None):
         state = np.zeros((H, d, e), F)
     o, state = gla_recurrence(q, k, v, gla_decay(z, mix["tau"]), state)
     o = rms_norm_plain(o, w[p + "norm"], eps).reshape(T, H * e)
-    return (o * silu(h @ w[p + "g"].T)) @ w[p + "o"].T, state
+    return rnd(o * silu(h @ w[p + "g"].T)) @ w[p + "o"].T, state
 
 
 def latent_rows(h, w, p, mix, eps, pos0):
@@ -110,23 +110,24 @@ def latent_attention(q, c, kr, uk, uv, sink, scale, size, pos0):
     return out
 
 
-def latent_mixer(h, w, p, mix, eps, past=None):
+def latent_mixer(h, w, p, mix, eps, past=None, rnd=lambda x: x):
     H, dim, rot, R, e, T = mix["heads"], mix["dim"], mix["rot_dim"], mix["kv_rank"], mix["vdim"], h.shape[0]
     pos0 = 0 if past is None else past[0].shape[0]
     q = (h @ w[p + "q"].T).reshape(T, H, dim + rot)
     for t in range(T):
         q[t, :, dim:] = rotate_interleaved(q[t, :, dim:], pos0 + t, mix["rot"]["base"], mix["rot"]["dims"])
-    c, kr = latent_rows(h, w, p, mix, eps, pos0)
+    q = rnd(q)
+    c, kr = map(rnd, latent_rows(h, w, p, mix, eps, pos0))
     if past is not None:
         c, kr = np.concatenate([past[0], c]), np.concatenate([past[1], kr])
     size = mix["mask"]["size"] if mix.get("mask") else None
     o = latent_attention(q, c, kr, w[p + "uk"].reshape(H, dim, R), w[p + "uv"].reshape(H, e, R), w[p + "sink"], mix["scale"], size, pos0)
-    o = o * sigmoid(h @ w[p + "g"].T)[:, :, None]
+    o = rnd(o * sigmoid(h @ w[p + "g"].T)[:, :, None])
     return o.reshape(T, H * e) @ w[p + "o"].T, (c, kr)
 
 
-def dense_ff(h, w, p):
-    return gelu_tanh(h @ w[p + "up"].T) @ w[p + "down"].T
+def dense_ff(h, w, p, rnd=lambda x: x):
+    return rnd(gelu_tanh(h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
 MIXERS = {"gla": gla_mixer, "latent_attention": latent_mixer}
@@ -144,10 +145,12 @@ def layer_runs(cfg):
 
 
 class Plain:
-    """One sequence.  feed(tokens) returns the logits of every token fed and keeps what later tokens need."""
+    """One sequence.  feed(tokens) returns the logits of every token fed and keeps what later tokens need.  rnd is applied to every
+    row that a reduced-precision implementation may round (what enters a matrix product, queries, cached rows): with it the
+    decoder tells how far rounding alone moves the logits."""
 
-    def __init__(self, cfg, weights):
-        self.cfg = cfg
+    def __init__(self, cfg, weights, rnd=lambda x: x):
+        self.cfg, self.rnd = cfg, rnd
         self.w = {k: np.asarray(v, dtype=F) for k, v in weights.items()}
         self.kept = {}
         self.residuals = []
@@ -160,10 +163,10 @@ class Plain:
             lay, p = cfg["layers"][i], f"l{i}."
             if begins:
                 x = x + w["loop.step"][t]
-            y, self.kept[run] = MIXERS[lay["type"]](rms_norm_around_zero(x, w[p + "norm1"], eps), w, p + "mix.", lay["mixer"], eps,
-                                                    self.kept.get(run))
+            y, self.kept[run] = MIXERS[lay["type"]](self.rnd(rms_norm_around_zero(x, w[p + "norm1"], eps)), w, p + "mix.", lay["mixer"], eps,
+                                                    self.kept.get(run), self.rnd)
             x = x + y
             if lay["mlp"]:
-                x = x + dense_ff(rms_norm_around_zero(x, w[p + "norm2"], eps), w, p + "mlp.")
+                x = x + dense_ff(self.rnd(rms_norm_around_zero(x, w[p + "norm2"], eps)), w, p + "mlp.", self.rnd)
             self.residuals.append(x.copy())
-        return rms_norm_around_zero(x, w["final.norm"], eps) @ w["head"].T
+        return self.rnd(rms_norm_around_zero(x, w["final.norm"], eps)) @ w["head"].T
