@@ -18,7 +18,7 @@ constexpr int64_t FEW_ROWS = 16;           // rows up to which activations stay 
 constexpr int64_t GLA_TOKENWISE = 16;      // rows per sequence up to which the recurrence runs token by token
 constexpr int64_t LATENT_FEW = 8;          // rows per sequence up to which attention reads the latents themselves
 constexpr int64_t SPLIT_KEYS = 32;         // keys a split of that attention is cut into
-constexpr int64_t SPLIT_CTAS = 296, SPLIT_HEADS = 16;
+constexpr int64_t SPLIT_CTAS = 296, SPLIT_HEADS = 8;
 
 enum LayerType { GLA, LATENT };
 struct Layer {

@@ -12,7 +12,7 @@ namespace b200 {
 
 namespace {
 
-constexpr int DV_WARPS = 8;
+constexpr int DV_WARPS = 4;
 
 template <typename W>
 struct WLoad;   // a lane's 16-byte piece of a weight row
@@ -34,10 +34,10 @@ struct WLoad<float> {
 
 // RPW weight rows per warp group, NCOL activation rows; wpr warps share a row group (pieces dealt out in turn)
 template <typename W, int RPW, int NCOL, bool VEC>
-__global__ void __launch_bounds__(DV_WARPS * 32)
+__global__ void __launch_bounds__(DV_WARPS * 32, NCOL == 1 ? 8 : 4)
 dense_rows_kernel(DenseMm d, int m0, int wpr) {
     constexpr int E = VEC ? WLoad<W>::E : 1;
-    constexpr int U = VEC ? (RPW >= 4 ? 2 : 4) : 4;
+    constexpr int U = 2;   // pieces per row in flight
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int groups = DV_WARPS / wpr, grp = warp / wpr, sub = warp % wpr;
@@ -156,7 +156,7 @@ int launch_rows(const DenseMm &d, int m0, bool vec, int sms, cudaStream_t s) {
     const int64_t rg = (d.n + RPW - 1) / RPW;
     int wpr = 1;
     const int64_t pieces = (d.k + (vec ? 32 * WLoad<W>::E : 32) - 1) / (vec ? 32 * WLoad<W>::E : 32);
-    while (wpr < DV_WARPS && rg * wpr < (int64_t)sms * 12 && pieces > 2 * wpr) wpr *= 2;
+    while (wpr < DV_WARPS && rg * wpr < (int64_t)sms * 24 && pieces > 2 * wpr) wpr *= 2;
     const int64_t groups = DV_WARPS / wpr, blocks = (rg + groups - 1) / groups;
     B200_REQUIRE(blocks < 0x7fffffffLL, "dense mat-mul: too many rows");
     return vec ? launch_pdl(dense_rows_kernel<W, RPW, NCOL, true>, dim3((unsigned)blocks), dim3(DV_WARPS * 32), 0, s, d, m0, wpr)

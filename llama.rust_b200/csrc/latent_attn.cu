@@ -6,7 +6,7 @@
 // Cells of a sequence's positions are listed in `tab` (segment field TAB0: its first entry, KEY0: that entry's position).
 // Few rows per sequence: Uk moves to the query's side, so that attention reads the cached rows themselves, once for all heads:
 //   latent_query_kernel    queries through Uk and rotated; the rows' own latents normed, rotated and stored (one more block per row)
-//   latent_decode_kernel   per (split of keys, 16 heads, row): running softmax over 32-key tiles in shared memory, F32 arithmetic
+//   latent_decode_kernel   per (split of keys, 8 heads, row): running softmax over 32-key tiles in shared memory, F32 arithmetic
 //   latent_value_kernel    splits and sink merged, Uv, gate
 // Many rows: keys and values expanded for every listed cell by one mat-mul, then
 //   latent_attn_mma_kernel  64 rows x 64-key tiles on mma.sync (BF16 operands, F32 scores and sums; a weight goes in as two BF16
@@ -21,7 +21,7 @@ enum { LSEG_ROW0 = 0, LSEG_ROWS = 1, LSEG_POS0 = 4, LSEG_TAB0 = 5, LSEG_KEY0 = 6
 namespace {
 
 constexpr int LT = 256;             // threads per block
-constexpr int LK = 32, LH = 16;     // keys per tile, heads per block of the few-rows kernel
+constexpr int LK = 32, LH = 8;      // keys per tile, heads (one per warp) per block of the few-rows kernel
 constexpr int LRB = 512;            // latent elements a block of it accumulates
 constexpr int LV_ROWS = 32;         // value rows per block of the merge
 constexpr int ERR_CELL = 2, ERR_POS = 3;
@@ -92,7 +92,7 @@ latent_query_kernel(LatentArgs a, int lanes, int *err) {
     pdl_trigger();
     pdl_wait();
     if (h == a.heads) {
-        store_row<T>(a, row, part, err);
+        if (blockIdx.z == 0) store_row<T>(a, row, part, err);
         return;
     }
     const float *q = a.proj + row * a.ldp + a.off_q + h * (a.dim + a.rot);
@@ -104,8 +104,8 @@ latent_query_kernel(LatentArgs a, int lanes, int *err) {
     __syncthreads();
     const int groups = LT / lanes, g = tid / lanes, l = tid % lanes;
     const T *uk = (const T *)a.ukv + (int64_t)h * a.dim * a.rank;
-    for (int r0 = 0; r0 < a.rank; r0 += lanes * VEC) {
-        const int r = r0 + l * VEC;
+    {
+        const int r0 = blockIdx.z * lanes * VEC, r = r0 + l * VEC;
         float acc[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; e++) acc[e] = 0.0f;
@@ -127,9 +127,13 @@ latent_query_kernel(LatentArgs a, int lanes, int *err) {
             for (int k = 0; k < groups; k++) v += red[k * lanes * VEC + i];
             out[r0 + i] = v;
         }
-        __syncthreads();
     }
-    for (int j = tid; j < a.rot; j += LT) out[a.rank + j] = rotated(q + a.dim, rope, a.rot_dims, j);
+    if (blockIdx.z == 0)
+        for (int j = tid; j < a.rot; j += LT) out[a.rank + j] = rotated(q + a.dim, rope, a.rot_dims, j);
+}
+
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
 }
 
 // the keys a row sees: positions [lo, hi]
@@ -149,7 +153,7 @@ latent_decode_kernel(LatentArgs a, int head_groups, int *err) {
     T *sk = (T *)l_raw;                                              // [LK][units] pieces
     float *sq = (float *)(l_raw + (size_t)LK * units * 16);          // [LH][qs]
     float *sp = sq + LH * qs;                                        // [LK][LH] weights
-    float *sm = sp + LK * LH, *sl = sm + LH, *scorr = sl + LH;       // running maximum, sum, this tile's correction
+    float *scorr = sp + LK * LH;                                     // [LH] what this tile's maximum makes of the sums so far
     const int split = blockIdx.x, h0 = (blockIdx.y % head_groups) * LH, rb0 = (blockIdx.y / head_groups) * LRB;
     const int64_t row = blockIdx.z;
     const int nh = min(LH, a.heads - h0);
@@ -164,36 +168,30 @@ latent_decode_kernel(LatentArgs a, int head_groups, int *err) {
         const int h = i / qs, d = i - h * qs;
         sq[i] = h < nh && d < D ? a.queries[(row * a.heads + h0 + h) * D + d] : 0.0f;
     }
-    if (tid < LH) {
-        sm[tid] = -INFINITY;
-        sl[tid] = 0.0f;
-    }
-    float acc[LH][2];
+    float acc[LH][2], m = -INFINITY, l = 0.0f;   // m, l: of the warp's head
 #pragma unroll
     for (int h = 0; h < LH; h++) acc[h][0] = acc[h][1] = 0.0f;
     const int r = rb0 + 2 * tid;
     for (int k0 = lo; k0 < hi; k0 += LK) {
         const int kn = min(LK, hi - k0);
         __syncthreads();
-        // rows of cells: 16-byte pieces (a cell's row is padded to whole ones)
-        for (int i = tid; i < LK * pieces; i += LT) {
-            const int k = i / pieces, p = i - k * pieces;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (k < kn) {
-                const int64_t at = tab0 + k0 + k;
-                const int64_t cell = at >= 0 && at < a.n_tab ? a.tab[at] : -1;
-                if (cell >= 0 && cell < a.n_cells) v = *reinterpret_cast<const uint4 *>((const T *)a.cache + cell * a.ldc + p * PE);
-                else if (p == 0) atomicExch(err, ERR_CELL);
-            }
-            *reinterpret_cast<uint4 *>(sk + ((size_t)k * units + p) * PE) = v;
+        // rows of cells, a warp four at a time: 16-byte pieces (a cell's row is padded to whole ones)
+        for (int k = warp; k < LK; k += LT / 32) {
+            const int64_t at = (int64_t)tab0 + k0 + k;
+            const int64_t cell = k < kn && at >= 0 && at < a.n_tab ? a.tab[at] : -1;
+            const bool in = cell >= 0 && cell < a.n_cells;
+            if (k < kn && !in && lane == 0) atomicExch(err, ERR_CELL);
+            const T *src = (const T *)a.cache + (in ? cell * a.ldc : 0);
+            for (int p = lane; p < pieces; p += 32) cp16(sk + ((size_t)k * units + p) * PE, src + p * PE, in);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        // scores: lane = key, two heads per warp
+        // scores: lane = key, warp = head
         {
-            const int ha = 2 * warp, hb = ha + 1;
             const T *kr = sk + (size_t)lane * units * PE;
-            const float *qa = sq + ha * qs, *qb = sq + hb * qs;
-            float s0 = 0.0f, s1 = 0.0f;
+            const float *qa = sq + warp * qs;
+            float s4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll 4
             for (int p = 0; p < pieces; p++) {
                 const uint4 w = *reinterpret_cast<const uint4 *>(kr + p * PE);
@@ -206,27 +204,19 @@ latent_decode_kernel(LatentArgs a, int head_groups, int *err) {
                 }
 #pragma unroll
                 for (int e = 0; e < PE; e += 4) {
-                    const float4 x = *reinterpret_cast<const float4 *>(qa + p * PE + e), y = *reinterpret_cast<const float4 *>(qb + p * PE + e);
-                    s0 = fmaf(x.x, f[e], fmaf(x.y, f[e + 1], fmaf(x.z, f[e + 2], fmaf(x.w, f[e + 3], s0))));
-                    s1 = fmaf(y.x, f[e], fmaf(y.y, f[e + 1], fmaf(y.z, f[e + 2], fmaf(y.w, f[e + 3], s1))));
+                    const float4 x = *reinterpret_cast<const float4 *>(qa + p * PE + e);
+                    s4[0] = fmaf(x.x, f[e], s4[0]);
+                    s4[1] = fmaf(x.y, f[e + 1], s4[1]);
+                    s4[2] = fmaf(x.z, f[e + 2], s4[2]);
+                    s4[3] = fmaf(x.w, f[e + 3], s4[3]);
                 }
             }
-#pragma unroll
-            for (int u = 0; u < 2; u++) {
-                const int h = ha + u;
-                const float s = lane < kn ? (u ? s1 : s0) * a.scale : -INFINITY;
-                const float mo = sm[h], mn = fmaxf(mo, warp_max(s));
-                const float p = lane < kn ? expf(s - mn) : 0.0f;
-                const float sum = warp_sum(p);
-                sp[lane * LH + h] = p;
-                __syncwarp();
-                if (lane == 0) {
-                    const float corr = mo == -INFINITY ? 0.0f : expf(mo - mn);
-                    scorr[h] = corr;
-                    sm[h] = mn;
-                    sl[h] = sl[h] * corr + sum;
-                }
-            }
+            const float s = lane < kn ? ((s4[0] + s4[1]) + (s4[2] + s4[3])) * a.scale : -INFINITY;
+            const float mn = fmaxf(m, warp_max(s)), corr = m == -INFINITY ? 0.0f : expf(m - mn), p = lane < kn ? expf(s - mn) : 0.0f;
+            l = l * corr + warp_sum(p);
+            m = mn;
+            sp[lane * LH + warp] = p;
+            if (lane == 0) scorr[warp] = corr;
         }
         __syncthreads();
         if (r < a.rank) {
@@ -267,16 +257,16 @@ latent_decode_kernel(LatentArgs a, int head_groups, int *err) {
         if (r < a.rank) out[(int64_t)h * (a.rank + 2) + r] = acc[h][0];
         if (r + 1 < a.rank) out[(int64_t)h * (a.rank + 2) + r + 1] = acc[h][1];
     }
-    if (rb0 == 0 && tid < nh) {
-        out[(int64_t)tid * (a.rank + 2) + a.rank] = sm[tid];
-        out[(int64_t)tid * (a.rank + 2) + a.rank + 1] = sl[tid];
+    if (rb0 == 0 && lane == 0 && warp < nh) {
+        out[(int64_t)warp * (a.rank + 2) + a.rank] = m;
+        out[(int64_t)warp * (a.rank + 2) + a.rank + 1] = l;
     }
 }
 
 template <typename T, typename Y, int VEC>
 __global__ void __launch_bounds__(LT)
 latent_value_kernel(LatentArgs a) {
-    extern __shared__ float l_sm[];   // [rank]
+    extern __shared__ float l_sm[];   // [rank], then [n_splits]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
     const int64_t row = blockIdx.y;
     pdl_trigger();
@@ -285,15 +275,26 @@ latent_value_kernel(LatentArgs a) {
     const int splits = min(a.n_splits, (keys + a.per_split - 1) / a.per_split);
     const int64_t step = (int64_t)a.heads * (a.rank + 2);
     const float *p = a.partial + (row * a.n_splits * a.heads + h) * (int64_t)(a.rank + 2);
-    float m = a.sink[h];
-    for (int s = 0; s < splits; s++) m = fmaxf(m, p[s * step + a.rank]);
-    float l = expf(a.sink[h] - m);
-    for (int s = 0; s < splits; s++) l = fmaf(p[s * step + a.rank + 1], expf(p[s * step + a.rank] - m), l);
-    const float inv = 1.0f / l;
+    float *sw = l_sm + (a.rank + 3) / 4 * 4;   // [splits] what each split counts
+    if (warp == 0) {
+        float m = a.sink[h];
+        for (int s = lane; s < splits; s += 32) m = fmaxf(m, p[s * step + a.rank]);
+        m = warp_max(m);
+        float l = 0.0f;
+        for (int s = lane; s < splits; s += 32) {
+            const float w = expf(p[s * step + a.rank] - m);
+            sw[s] = w;
+            l = fmaf(p[s * step + a.rank + 1], w, l);
+        }
+        l = 1.0f / (warp_sum(l) + expf(a.sink[h] - m));
+        for (int s = lane; s < splits; s += 32) sw[s] *= l;
+    }
+    __syncthreads();
     for (int r = tid; r < a.rank; r += LT) {
         float v = 0.0f;
-        for (int s = 0; s < splits; s++) v = fmaf(p[s * step + r], expf(p[s * step + a.rank] - m), v);
-        l_sm[r] = v * inv;
+#pragma unroll 8
+        for (int s = 0; s < splits; s++) v = fmaf(p[s * step + r], sw[s], v);
+        l_sm[r] = v;
     }
     __syncthreads();
     const float gate = sigmoid_f32(a.proj[row * a.ldp + a.off_g + h]);
@@ -398,19 +399,18 @@ __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
 __device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void *p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
 }
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
 
 constexpr int MT = 128, MQ = 64, MK = 64;
 
+// One buffer each for keys and values: the next keys land while the weights meet the values, the next values while the queries meet
+// the keys; three blocks per SM cover each other's waits.
 template <typename Y, int DK, int DV, bool ALIGNED>
-__global__ void __launch_bounds__(MT)
+__global__ void __launch_bounds__(MT, DK <= 192 ? 3 : 2)
 latent_attn_mma_kernel(LatentArgs a, int *err) {
     typedef __nv_bfloat16 bf;
     constexpr int KS = DK + 8, VS = DV + 8;   // row strides: an odd number of 16-byte units
     extern __shared__ __align__(16) uint8_t l_raw[];
-    bf *sQ = (bf *)l_raw, *sK = sQ + MQ * KS, *sV = sK + 2 * MK * KS;   // two stages of keys and values
+    bf *sQ = (bf *)l_raw, *sK = sQ + MQ * KS, *sV = sK + MK * KS;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, D = a.dim + a.rot;
     pdl_trigger();
     pdl_wait();
@@ -426,42 +426,55 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
         return;
     }
     const int tiles = (last - lo) / MK + 1;
-    const bf *kvp = (const bf *)a.kv, *rp = (const bf *)a.cache;
-    const auto load_tile = [&](int t) {
-        bf *k = sK + (t & 1) * MK * KS, *v = sV + (t & 1) * MK * VS;
-        const int k0 = lo + t * MK;
-        if constexpr (ALIGNED) {
-            constexpr int KP = DK / 8, VP = DV / 8;
-            const int np = a.dim / 8, dp = D / 8, vp = a.vdim / 8;
-            for (int i = tid; i < MK * KP; i += MT) {
-                const int j = i / KP, p = i - j * KP;
-                const bool in = k0 + j <= last && p < dp;
-                const int64_t at = base + (k0 + j <= last ? k0 + j : lo);
-                const bf *src = p < np ? kvp + at * a.ldkv + h * a.dim + p * 8 : rp + at * a.ldc + a.rank + (p < dp ? p - np : 0) * 8;
-                cp16(k + j * KS + p * 8, src, in);
-            }
-            for (int i = tid; i < MK * VP; i += MT) {
-                const int j = i / VP, p = i - j * VP;
-                const bool in = k0 + j <= last && p < vp;
-                const int64_t at = base + (k0 + j <= last ? k0 + j : lo);
-                cp16(v + j * VS + p * 8, kvp + at * a.ldkv + a.heads * a.dim + h * a.vdim + (p < vp ? p : 0) * 8, in);
-            }
-        } else {
-            const bf zero = __float2bfloat16_rn(0.0f);
-            for (int i = tid; i < MK * DK; i += MT) {
-                const int j = i / DK, d = i - j * DK;
-                bf x = zero;
-                if (k0 + j <= last && d < D) x = d < a.dim ? kvp[(base + k0 + j) * a.ldkv + h * a.dim + d] : rp[(base + k0 + j) * a.ldc + a.rank + d - a.dim];
-                k[j * KS + d] = x;
-            }
-            for (int i = tid; i < MK * DV; i += MT) {
-                const int j = i / DV, c = i - j * DV;
-                v[j * VS + c] = k0 + j <= last && c < a.vdim ? kvp[(base + k0 + j) * a.ldkv + a.heads * a.dim + h * a.vdim + c] : zero;
+    const bf *kn = (const bf *)a.kv + (base + lo) * a.ldkv + h * a.dim, *kr = (const bf *)a.cache + (base + lo) * a.ldc + a.rank;
+    const bf *vp = (const bf *)a.kv + (base + lo) * a.ldkv + a.heads * a.dim + h * a.vdim;
+    const int ldkv = (int)a.ldkv, ldc = (int)a.ldc;
+    // key j of the sequence stands at lo + j; rows past the last key and channels past the head's are zero
+    const auto load_keys = [&](int t) {
+        const int j0 = t * MK, jn = last - lo - j0;   // keys 0 .. jn of the tile exist
+        if (t < tiles) {
+            if constexpr (ALIGNED) {
+                constexpr int KP = DK / 8;
+                const int np = a.dim / 8, dp = D / 8;
+                for (int i = tid; i < MK * KP; i += MT) {
+                    const int j = i / KP, p = i - j * KP;
+                    const bool in = j <= jn && p < dp;
+                    const int at = in ? j0 + j : 0, q = in ? p : 0;
+                    cp16(sK + j * KS + p * 8, q < np ? kn + (int64_t)at * ldkv + q * 8 : kr + (int64_t)at * ldc + (q - np) * 8, in);
+                }
+            } else {
+                for (int i = tid; i < MK * DK; i += MT) {
+                    const int j = i / DK, d = i - j * DK;
+                    bf x = __float2bfloat16_rn(0.0f);
+                    if (j <= jn && d < D) x = d < a.dim ? kn[(int64_t)(j0 + j) * ldkv + d] : kr[(int64_t)(j0 + j) * ldc + d - a.dim];
+                    sK[j * KS + d] = x;
+                }
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    load_tile(0);
+    const auto load_values = [&](int t) {
+        const int j0 = t * MK, jn = last - lo - j0;
+        if (t < tiles) {
+            if constexpr (ALIGNED) {
+                constexpr int VP = DV / 8;
+                const int np = a.vdim / 8;
+                for (int i = tid; i < MK * VP; i += MT) {
+                    const int j = i / VP, p = i - j * VP;
+                    const bool in = j <= jn && p < np;
+                    cp16(sV + j * VS + p * 8, vp + (in ? (int64_t)(j0 + j) * ldkv + p * 8 : 0), in);
+                }
+            } else {
+                for (int i = tid; i < MK * DV; i += MT) {
+                    const int j = i / DV, c = i - j * DV;
+                    sV[j * VS + c] = j <= jn && c < a.vdim ? vp[(int64_t)(j0 + j) * ldkv + c] : __float2bfloat16_rn(0.0f);
+                }
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load_keys(0);
+    load_values(0);
     for (int i = tid; i < MQ * DK; i += MT) {
         const int t = i / DK, d = i - t * DK;
         float x = 0.0f;
@@ -478,48 +491,58 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
     for (int i = 0; i < DV / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const float sc = a.scale * 1.4426950408889634f;   // powers of two
     const int window = a.window > 0 ? a.window : 0x7fffffff;
+    const bf *qp = sQ + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8;
+    const bf *kp = sK + ((lane >> 4) * 8 + (lane & 7)) * KS + ((lane >> 3) & 1) * 8;
+    const bf *vq = sV + (((lane >> 3) & 1) * 8 + (lane & 7)) * VS + (lane >> 4) * 8;
     for (int t = 0; t < tiles; t++) {
-        if (t + 1 < tiles) {
-            load_tile(t + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const bf *k = sK + (t & 1) * MK * KS, *v = sV + (t & 1) * MK * VS;
         const int k0 = lo + t * MK;
+        asm volatile("cp.async.wait_group 1;" ::: "memory");   // the keys; the values may still be on their way
+        __syncthreads();
         float s[MK / 8][4];
 #pragma unroll
         for (int i = 0; i < MK / 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
 #pragma unroll
         for (int kk = 0; kk < DK / 16; kk++) {
             uint32_t qa[4];
-            ldsm4(qa, sQ + (warp * 16 + (lane & 15)) * KS + kk * 16 + (lane >> 4) * 8);
+            ldsm4(qa, qp + kk * 16);
 #pragma unroll
             for (int j = 0; j < MK / 16; j++) {
                 uint32_t kb[4];   // keys 16 j .. + 7 and + 8 .. + 15, both halves of the 16 channels
-                ldsm4(kb, k + (j * 16 + (lane >> 4) * 8 + (lane & 7)) * KS + kk * 16 + ((lane >> 3) & 1) * 8);
+                ldsm4(kb, kp + j * 16 * KS + kk * 16);
                 mma_bf16(s[2 * j], qa, kb[0], kb[1]);
                 mma_bf16(s[2 * j + 1], qa, kb[2], kb[3]);
             }
         }
+        __syncthreads();
+        load_keys(t + 1);
+        // powers of two of the scaled scores; only tiles at an edge of what the rows see need the mask
         float mx[2] = {m[0], m[1]};
+        if (k0 + MK - 1 > pos0 || pos0 + MQ - 1 - k0 >= window) {
 #pragma unroll
-        for (int i = 0; i < MK / 8; i++) {
+            for (int i = 0; i < MK / 8; i++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int key = k0 + i * 8 + 2 * (lane & 3) + (e & 1), p = e < 2 ? pa : pb;
-                s[i][e] = key <= p && p - key < window ? s[i][e] * sc : -INFINITY;
-                mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
-            }
+                for (int e = 0; e < 4; e++) {
+                    const int key = k0 + i * 8 + 2 * (lane & 3) + (e & 1), p = e < 2 ? pa : pb;
+                    s[i][e] = key <= p && p - key < window ? s[i][e] * sc : -INFINITY;
+                    mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
+                }
+        } else {
+#pragma unroll
+            for (int i = 0; i < MK / 8; i++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    s[i][e] *= sc;
+                    mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
+                }
         }
-        float corr[2];
+        float corr[2], mm[2];
 #pragma unroll
         for (int u = 0; u < 2; u++) {
             mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffffu, mx[u], 1));
             mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffffu, mx[u], 2));
             corr[u] = m[u] == -INFINITY ? 0.0f : exp2f(m[u] - mx[u]);
             m[u] = mx[u];
+            mm[u] = mx[u] == -INFINITY ? 0.0f : mx[u];   // a row that has seen nothing yet: every power below is of minus infinity
             l[u] *= corr[u];
         }
 #pragma unroll
@@ -529,30 +552,38 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
             o[i][2] *= corr[1];
             o[i][3] *= corr[1];
         }
+        asm volatile("cp.async.wait_group 1;" ::: "memory");   // the values; the next keys may still be on their way
+        __syncthreads();
 #pragma unroll
         for (int j = 0; j < MK / 16; j++) {
             uint32_t ph[4], pl[4];
 #pragma unroll
             for (int u = 0; u < 4; u++) {   // fragment registers: (rows a, keys low), (rows b, low), (a, high), (b, high)
                 const int i = 2 * j + (u >> 1), e = 2 * (u & 1);
-                const float mm = m[u & 1];
-                const float x = mm == -INFINITY ? 0.0f : exp2f(s[i][e] - mm), y = mm == -INFINITY ? 0.0f : exp2f(s[i][e + 1] - mm);
+                const float x = exp2f(s[i][e] - mm[u & 1]), y = exp2f(s[i][e + 1] - mm[u & 1]);
                 l[u & 1] += x + y;
                 ph[u] = bf16_pack(x, y);
                 pl[u] = bf16_pack(x - bf16_lo(ph[u]), y - bf16_hi(ph[u]));
             }
 #pragma unroll
-            for (int c = 0; c < DV / 16; c++) {
-                uint32_t vb[4];
-                ldsm4_t(vb, v + (j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * VS + c * 16 + (lane >> 4) * 8);
-                mma_bf16(o[2 * c], ph, vb[0], vb[1]);
-                mma_bf16(o[2 * c], pl, vb[0], vb[1]);
-                mma_bf16(o[2 * c + 1], ph, vb[2], vb[3]);
-                mma_bf16(o[2 * c + 1], pl, vb[2], vb[3]);
+            for (int c = 0; c < DV / 16; c += 2) {
+                uint32_t va[4], vb[4];
+                ldsm4_t(va, vq + j * 16 * VS + c * 16);
+                ldsm4_t(vb, vq + j * 16 * VS + c * 16 + 16);
+                mma_bf16(o[2 * c], ph, va[0], va[1]);
+                mma_bf16(o[2 * c + 1], ph, va[2], va[3]);
+                mma_bf16(o[2 * c + 2], ph, vb[0], vb[1]);
+                mma_bf16(o[2 * c + 3], ph, vb[2], vb[3]);
+                mma_bf16(o[2 * c], pl, va[0], va[1]);
+                mma_bf16(o[2 * c + 1], pl, va[2], va[3]);
+                mma_bf16(o[2 * c + 2], pl, vb[0], vb[1]);
+                mma_bf16(o[2 * c + 3], pl, vb[2], vb[3]);
             }
         }
-        __syncthreads();   // the stage is free for the tile after next
+        __syncthreads();
+        load_values(t + 1);
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     const float sink = a.sink[h] * 1.4426950408889634f;
 #pragma unroll
     for (int u = 0; u < 2; u++) {
@@ -589,17 +620,20 @@ int allow_smem(K kernel, size_t smem) {
 
 template <typename T, int VEC>
 int run_query(const LatentArgs &a, int *err, cudaStream_t s) {
+    // a block takes 16 pieces of the rank: enough blocks for one row
     int lanes = 1;
-    while (lanes < LT && lanes * VEC < a.rank) lanes *= 2;
+    while (lanes < 16 && lanes * VEC < a.rank) lanes *= 2;
+    const unsigned blocks = (unsigned)((a.rank + lanes * VEC - 1) / (lanes * VEC));
+    B200_REQUIRE(blocks <= 65535, "latent attention: rank %d is too large", a.rank);
     const size_t smem = ((size_t)(a.dim + 3) / 4 * 4 + (size_t)LT * VEC) * 4;
     int rc = allow_smem(latent_query_kernel<T, VEC>, smem);
     if (rc != B200_STATUS_SUCCESS) return rc;
-    return launch_pdl(latent_query_kernel<T, VEC>, dim3((unsigned)a.heads + 1, (unsigned)a.n), dim3(LT), smem, s, a, lanes, err);
+    return launch_pdl(latent_query_kernel<T, VEC>, dim3((unsigned)a.heads + 1, (unsigned)a.n, blocks), dim3(LT), smem, s, a, lanes, err);
 }
 template <typename T>
 int run_decode(const LatentArgs &a, int *err, cudaStream_t s) {
     const int D = a.rank + a.rot, pe = 16 / (int)sizeof(T), qs = (D + pe - 1) / pe * pe;
-    const size_t smem = (size_t)LK * key_units<T>(D) * 16 + ((size_t)LH * qs + LK * LH + 3 * LH) * 4;
+    const size_t smem = (size_t)LK * key_units<T>(D) * 16 + ((size_t)LH * qs + LK * LH + LH) * 4;
     int rc = allow_smem(latent_decode_kernel<T>, smem);
     if (rc != B200_STATUS_SUCCESS) return rc;
     const int hg = (a.heads + LH - 1) / LH, rb = (a.rank + LRB - 1) / LRB;
@@ -608,7 +642,7 @@ int run_decode(const LatentArgs &a, int *err, cudaStream_t s) {
 template <typename T, int VEC>
 int run_value(const LatentArgs &a, cudaStream_t s) {
     const dim3 g((unsigned)a.heads, (unsigned)a.n, (unsigned)((a.vdim + LV_ROWS - 1) / LV_ROWS));
-    const size_t smem = (size_t)a.rank * 4 + 64;
+    const size_t smem = ((size_t)a.rank + 4 + a.n_splits) * 4;
     if (a.y_type == B200_TYPE_F32) {
         int rc = allow_smem(latent_value_kernel<T, float, VEC>, smem);
         return rc != B200_STATUS_SUCCESS ? rc : launch_pdl(latent_value_kernel<T, float, VEC>, g, dim3(LT), smem, s, a);
@@ -625,7 +659,7 @@ int run_attn_any(const LatentArgs &a, int *err, cudaStream_t s) {
 }
 template <typename Y, int DK, int DV, bool ALIGNED>
 int run_attn_mma(const LatentArgs &a, int *err, cudaStream_t s) {
-    const size_t smem = ((size_t)MQ * (DK + 8) + 2 * (size_t)MK * (DK + 8 + DV + 8)) * 2;
+    const size_t smem = ((size_t)MQ * (DK + 8) + (size_t)MK * (DK + 8 + DV + 8)) * 2;
     int rc = allow_smem(latent_attn_mma_kernel<Y, DK, DV, ALIGNED>, smem);
     if (rc != B200_STATUS_SUCCESS) return rc;
     return launch_pdl(latent_attn_mma_kernel<Y, DK, DV, ALIGNED>, dim3((unsigned)((a.n + MQ - 1) / MQ + a.n_seg), (unsigned)a.heads), dim3(MT), smem, s, a, err);
