@@ -22,6 +22,10 @@ __device__ __forceinline__ uint32_t bf16_pack(float lo, float hi) {
     return *reinterpret_cast<const uint32_t *>(&v);
 }
 
+// ask L2 for a line: a kernel does it ahead of pdl_wait() for what it will read (nothing is read here, so it may be something that
+// an earlier kernel still writes)
+__device__ __forceinline__ void l2_prefetch(const void *p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -44,12 +44,17 @@ gla_step_kernel(GlaArgs a, int lanes, int cols) {
     const int groups = GLA_THREADS / lanes, grp = tid / lanes, c0 = (tid % lanes) * VEC;
     float *s_a = gla_sm, *s_k = s_a + a.dim, *s_q = s_k + a.dim, *s_red = s_q + a.dim;   // s_red [groups][cols]
     pdl_trigger();
-    pdl_wait();
+    // the step's inputs are in place before its first kernel starts
     const int32_t *sg = a.seg + (int64_t)blockIdx.z * GSEG_FIELDS;
     const int row0 = sg[GSEG_ROW0], rows = sg[GSEG_ROWS];
     bool fresh = sg[GSEG_FRESH] != 0;
     float *S = a.state + (((int64_t)sg[GSEG_SLOT] * a.heads + h) * a.dim) * a.vdim + v0;
     const W *a2 = (const W *)a.a2 + (int64_t)h * a.dim * a.rank;
+    for (int d = tid; d < a.dim; d += GLA_THREADS) {
+        for (int c = 0; c < vn; c += 32) l2_prefetch(S + (int64_t)d * a.vdim + c);
+        l2_prefetch(a2 + (int64_t)d * a.rank);
+    }
+    pdl_wait();
     const bool active = c0 < vn;
     for (int t = 0; t < rows; t++) {
         const float *p = a.proj + (int64_t)(row0 + t) * a.ldp;
@@ -175,13 +180,13 @@ gla_chunk_kernel(GlaArgs a, GlaScratch sc) {
     const int64_t ch = (int64_t)ci * a.heads + h;
 
     // q and k; what pads a row is zero (decays: one)
-    for (int i = tid; i < C * (DP / VEC); i += GLA_THREADS) {
-        const int t = i / (DP / VEC), d = (i - t * (DP / VEC)) * VEC;
-        const bool in = t < rows && d < dim;
-        const float *p = proj + (in ? (int64_t)t * a.ldp + h * dim + d : 0);
-        gla_cp<4 * VEC>(sQ + t * DP + d, p + a.off_q, in);
-        gla_cp<4 * VEC>(sK + t * DP + d, p + a.off_k, in);
-    }
+    for (int t = warp; t < C; t += GLA_THREADS / 32)
+        for (int d = lane * VEC; d < DP; d += 32 * VEC) {
+            const bool in = t < rows && d < dim;
+            const float *p = proj + (in ? (int64_t)t * a.ldp + h * dim + d : 0);
+            gla_cp<4 * VEC>(sQ + t * DP + d, p + a.off_q, in);
+            gla_cp<4 * VEC>(sK + t * DP + d, p + a.off_k, in);
+        }
     asm volatile("cp.async.commit_group;" ::: "memory");
     for (int i = tid; i < C * (DP - dim); i += GLA_THREADS) sD[i / (DP - dim) * DP + dim + i % (DP - dim)] = 1.0f;
     for (int i = tid; i < NB * (DP - dim); i += GLA_THREADS) sT[i / (DP - dim) * DP + dim + i % (DP - dim)] = 1.0f;
@@ -288,24 +293,32 @@ gla_chunk_kernel(GlaArgs a, GlaScratch sc) {
         for (int J = 0; J < NB; J++)
             if (J < I) A[(J * GLA_SUB + j) * C + I * GLA_SUB + i] = acc[J];
         __syncthreads();
-        for (int e = tid; e < I * GLA_SUB * (DP / 4); e += GLA_THREADS) {
-            const int t = e / (DP / 4), d = (e - t * (DP / 4)) * 4;
-            float4 *k = reinterpret_cast<float4 *>(sK + t * DP + d);
-            const float4 w = *reinterpret_cast<const float4 *>(sT + I * DP + d), v = *k;
-            *k = make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w);
+        for (int d = lane * 4; d < DP; d += 128) {
+            const float4 w = *reinterpret_cast<const float4 *>(sT + I * DP + d);
+            for (int t = warp; t < I * GLA_SUB; t += GLA_THREADS / 32) {
+                float4 *k = reinterpret_cast<float4 *>(sK + t * DP + d);
+                const float4 v = *k;
+                *k = make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w);
+            }
         }
         __syncthreads();
     }
     // out: keys at the chunk's end, queries at its start (transposed), the chunk's decay
-    for (int i = tid; i < C * dim; i += GLA_THREADS) {
-        const int t = i / dim, d = i - t * dim;
-        sc.k[ch * C * dim + i] = sK[t * DP + d];
-    }
-    for (int i = tid; i < C * dim; i += GLA_THREADS) {
-        const int d = i / C, t = i % C;
-        float v = sQ[t * DP + d];
-        for (int s = t / GLA_SUB - 1; s >= 0; s--) v *= sT[s * DP + d];
-        sc.q[ch * C * dim + i] = v;
+    for (int t = warp; t < C; t += GLA_THREADS / 32)
+        for (int d = lane * VEC; d < dim; d += 32 * VEC) {
+            float *p = sc.k + ch * C * dim + t * dim + d;
+            if constexpr (VEC == 4) *reinterpret_cast<float4 *>(p) = *reinterpret_cast<const float4 *>(sK + t * DP + d);
+            else *p = sK[t * DP + d];
+        }
+    // (a thread: one channel, every 16th token's block in turn, so that the decay in front of a block is carried along)
+    for (int i = tid; i < GLA_SUB * dim; i += GLA_THREADS) {
+        const int d = i / GLA_SUB, t = i % GLA_SUB;
+        float w = 1.0f;
+#pragma unroll
+        for (int s = 0; s < NB; s++) {
+            sc.q[ch * C * dim + d * C + s * GLA_SUB + t] = sQ[(s * GLA_SUB + t) * DP + d] * w;
+            w *= sT[s * DP + d];
+        }
     }
     for (int d = tid; d < dim; d += GLA_THREADS) {
         float v = 1.0f;

@@ -90,6 +90,12 @@ latent_query_kernel(LatentArgs a, int lanes, int *err) {
     const int tid = threadIdx.x, h = blockIdx.x;
     const int64_t row = blockIdx.y;
     pdl_trigger();
+    if (h < a.heads) {
+        // this block's columns of the head's key rows
+        const int r0 = blockIdx.z * lanes * VEC, lines = (min(lanes * VEC, a.rank - r0) * (int)sizeof(T) + 127) / 128;
+        const T *uk = (const T *)a.ukv + (int64_t)h * a.dim * a.rank + r0;
+        for (int i = tid; i < a.dim * lines; i += LT) l2_prefetch((const char *)(uk + (int64_t)(i / lines) * a.rank) + 128 * (i % lines));
+    }
     pdl_wait();
     if (h == a.heads) {
         if (blockIdx.z == 0) store_row<T>(a, row, part, err);
@@ -269,7 +275,13 @@ latent_value_kernel(LatentArgs a) {
     extern __shared__ float l_sm[];   // [rank], then [n_splits]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
     const int64_t row = blockIdx.y;
+    const T *uv = (const T *)a.ukv + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim) * a.rank;
     pdl_trigger();
+    {
+        const int e0 = blockIdx.z * LV_ROWS, en = min(a.vdim, e0 + LV_ROWS);
+        const char *w0 = (const char *)(uv + (int64_t)e0 * a.rank), *w1 = (const char *)(uv + (int64_t)en * a.rank);
+        for (const char *w = w0 + 128 * tid; w < w1; w += 128 * LT) l2_prefetch(w);
+    }
     pdl_wait();
     const int pos = a.pos[row], keys = pos + 1 - first_key(a, pos);
     const int splits = min(a.n_splits, (keys + a.per_split - 1) / a.per_split);
@@ -298,7 +310,6 @@ latent_value_kernel(LatentArgs a) {
     }
     __syncthreads();
     const float gate = sigmoid_f32(a.proj[row * a.ldp + a.off_g + h]);
-    const T *uv = (const T *)a.ukv + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim) * a.rank;
     for (int e = blockIdx.z * LV_ROWS + warp; e < min(a.vdim, (int)(blockIdx.z + 1) * LV_ROWS); e += LT / 32) {
         const T *w = uv + (int64_t)e * a.rank;
         float acc = 0.0f;
@@ -415,7 +426,8 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
     pdl_trigger();
     pdl_wait();
     int r0, rows;
-    const int32_t *sg = find_tile(a, MQ, blockIdx.x, &r0, &rows);
+    // later tiles of a prompt see more keys: they go first
+    const int32_t *sg = find_tile(a, MQ, gridDim.x - 1 - blockIdx.x, &r0, &rows);
     if (!sg) return;
     const int64_t row0 = sg[LSEG_ROW0] + r0;
     const int pos0 = sg[LSEG_POS0] + r0, last = pos0 + rows - 1;
@@ -475,14 +487,33 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
     };
     load_keys(0);
     load_values(0);
-    for (int i = tid; i < MQ * DK; i += MT) {
-        const int t = i / DK, d = i - t * DK;
-        float x = 0.0f;
-        if (t < rows && d < D) {
-            const float *q = a.proj + (row0 + t) * a.ldp + a.off_q + h * D;
-            x = d < a.dim ? q[d] : rotated(q + a.dim, a.rope + (int64_t)(pos0 + t) * a.rot_dims, a.rot_dims, d - a.dim);
+    if constexpr (ALIGNED) {
+        // four channels at a time (two pairs of a rotated part), several pieces in flight
+        constexpr int QP = DK / 4;
+#pragma unroll 4
+        for (int i = tid; i < MQ * QP; i += MT) {
+            const int t = i / QP, d = (i - t * QP) * 4;
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (t < rows && d < D) {
+                x = *reinterpret_cast<const float4 *>(a.proj + (row0 + t) * a.ldp + a.off_q + h * D + d);
+                const int j = d - a.dim;
+                if (j >= 0 && j < a.rot_dims) {
+                    const float4 w = *reinterpret_cast<const float4 *>(a.rope + (int64_t)(pos0 + t) * a.rot_dims + j);   // cos, sin, cos, sin
+                    x = make_float4(fmaf(x.x, w.x, -(x.y * w.y)), fmaf(x.y, w.x, x.x * w.y), fmaf(x.z, w.z, -(x.w * w.w)), fmaf(x.w, w.z, x.z * w.w));
+                }
+            }
+            *reinterpret_cast<uint2 *>(sQ + t * KS + d) = make_uint2(bf16_pack(x.x, x.y), bf16_pack(x.z, x.w));
         }
-        sQ[t * KS + d] = __float2bfloat16_rn(x);
+    } else {
+        for (int i = tid; i < MQ * DK; i += MT) {
+            const int t = i / DK, d = i - t * DK;
+            float x = 0.0f;
+            if (t < rows && d < D) {
+                const float *q = a.proj + (row0 + t) * a.ldp + a.off_q + h * D;
+                x = d < a.dim ? q[d] : rotated(q + a.dim, a.rope + (int64_t)(pos0 + t) * a.rot_dims, a.rot_dims, d - a.dim);
+            }
+            sQ[t * KS + d] = __float2bfloat16_rn(x);
+        }
     }
     // this lane's two rows of the warp's 16
     const int ra = warp * 16 + (lane >> 2), rb = ra + 8, pa = pos0 + ra, pb = pos0 + rb;
@@ -668,7 +699,7 @@ template <typename Y>
 int run_attn_bf16(const LatentArgs &a, int *err, cudaStream_t s) {
     const int D = a.dim + a.rot;
     const bool al = a.dim % 8 == 0 && a.rot % 8 == 0 && a.vdim % 8 == 0 && a.rank % 8 == 0 && a.ldkv % 8 == 0 && a.ldc % 8 == 0 &&
-                    (((uintptr_t)a.kv | (uintptr_t)a.cache) & 15) == 0;
+                    a.ldp % 4 == 0 && a.off_q % 4 == 0 && a.rot_dims % 4 == 0 && (((uintptr_t)a.kv | (uintptr_t)a.cache | (uintptr_t)a.proj | (uintptr_t)a.rope) & 15) == 0;
     if (D <= 128 && a.vdim <= 64) return al ? run_attn_mma<Y, 128, 64, true>(a, err, s) : run_attn_mma<Y, 128, 64, false>(a, err, s);
     if (D <= 192 && a.vdim <= 128) return al ? run_attn_mma<Y, 192, 128, true>(a, err, s) : run_attn_mma<Y, 192, 128, false>(a, err, s);
     if (D <= 256 && a.vdim <= 128) return al ? run_attn_mma<Y, 256, 128, true>(a, err, s) : run_attn_mma<Y, 256, 128, false>(a, err, s);
