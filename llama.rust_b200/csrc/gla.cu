@@ -228,32 +228,41 @@ gla_chunk_kernel(GlaArgs a, GlaScratch sc) {
     asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();
 
-    // A inside the 16-token blocks: a warp per column j, its key carried on token by token
+    // A inside the 16-token blocks: half a warp per column j, its key carried on token by token, four channels at a time
     float *A = sc.A + ch * C * C;
-    for (int col = warp; col < C; col += GLA_THREADS / 32) {
-        const int sb = col / GLA_SUB, j = col % GLA_SUB;
+    for (int pair = warp; pair < C / 2; pair += GLA_THREADS / 32) {
+        const int col = 2 * pair + (lane >> 4), l16 = lane & 15, sb = col / GLA_SUB, j = col % GLA_SUB, j0 = j & ~1;
         float acc[GLA_SUB];
 #pragma unroll
         for (int i = 0; i < GLA_SUB; i++) acc[i] = 0.0f;
-        for (int d = lane; d < dim; d += 32) {
-            float k = sK[col * DP + d];
+        for (int d = 4 * l16; d < DP - 4; d += 64) {   // what pads a row is a zero query and key
+            float4 k = *reinterpret_cast<const float4 *>(sK + col * DP + d);
 #pragma unroll
             for (int i = 0; i < GLA_SUB; i++) {
-                if (i < j) continue;
+                if (i < j0) continue;
                 const int at = (sb * GLA_SUB + i) * DP + d;
-                if (i > j) k *= sD[at];
-                acc[i] = fmaf(sQ[at], k, acc[i]);
+                if (i > j0) {
+                    float4 w = *reinterpret_cast<const float4 *>(sD + at);
+                    if (i == j) w = make_float4(1.0f, 1.0f, 1.0f, 1.0f);   // the pair's second column, at its own token
+                    k = make_float4(k.x * w.x, k.y * w.y, k.z * w.z, k.w * w.w);
+                }
+                const float4 q = *reinterpret_cast<const float4 *>(sQ + at);
+                acc[i] = fmaf(q.x, k.x, fmaf(q.y, k.y, fmaf(q.z, k.z, fmaf(q.w, k.w, acc[i]))));
             }
         }
-        float mine = 0.0f;
+        // 16 sums over 16 lanes: each step halves both, lane i ends with row i
 #pragma unroll
-        for (int i = 0; i < GLA_SUB; i++) {
-            const float v = warp_sum(acc[i]);
-            if (lane == i) mine = v;
+        for (int o = GLA_SUB / 2; o > 0; o >>= 1) {
+            const bool up = (l16 & o) != 0;
+#pragma unroll
+            for (int i = 0; i < o; i++) {
+                const float keep = up ? acc[i + o] : acc[i], send = up ? acc[i] : acc[i + o];
+                acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
         }
-        // the column: zero above its token, these 16 rows, and the rows below from the other blocks
-        for (int i = lane; i < sb * GLA_SUB; i += 32) A[col * C + i] = 0.0f;
-        if (lane < GLA_SUB) A[col * C + sb * GLA_SUB + lane] = lane >= j ? mine * a.q_factor : 0.0f;
+        // the column: zero above its token, these 16 rows; the rows below come from the other blocks
+        for (int i = l16; i < sb * GLA_SUB; i += 16) A[col * C + i] = 0.0f;
+        A[col * C + sb * GLA_SUB + l16] = l16 >= j ? acc[0] * a.q_factor : 0.0f;
     }
     __syncthreads();
     // q carries the decay since its block's start, k the decay to its block's end

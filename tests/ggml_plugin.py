@@ -5,9 +5,9 @@ import ctypes as C
 
 import numpy as np
 
-F32, F16, I32 = 0, 1, 26
+F32, F16, I32, BF16 = 0, 1, 26, 30
 OP_NONE, OP_ADD, OP_MUL_MAT, OP_MUL_MAT_ID, OP_FLASH_ATTN_EXT, OP_VIEW = 0, 2, 29, 30, 74, 37
-TYPE_TRAITS = {0: (1, 4), 1: (1, 2), 2: (32, 18), 8: (32, 34), 12: (256, 144), 14: (256, 210), 26: (1, 4), 27: (1, 8),
+TYPE_TRAITS = {0: (1, 4), 1: (1, 2), 2: (32, 18), 8: (32, 34), 12: (256, 144), 14: (256, 210), 26: (1, 4), 27: (1, 8), 30: (1, 2),
                39: (32, 17)}
 
 vp, sz = C.c_void_p, C.c_size_t
