@@ -1,6 +1,7 @@
-// Gated linear attention: per head a state S [dim][vdim] in F32 with
-//     S_t = diag(a_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   a_t = sigmoid(decay logit)^(1 / tau)  per key channel,
-// each head's o then RMS-normed over vdim, weighted, and multiplied by silu(g).  All of it in F32.
+// Gated linear attention: a head keeps a state S [dim][vdim]; a token first fades it, row d by its decay a[d] (the decay logit's
+// sigmoid to the power 1 / tau), then adds its key times its value, and reads it with its query:
+//     S[d][e] <- a[d] S[d][e] + k[d] v[e],      o[e] = sum_d q[d] S[d][e]
+// The head's o goes through an RMS norm with a weight and is gated by silu(g).  All of it in F32.
 //
 // Two forms.  Token by token (decode steps, short stretches): one launch, the value columns of a head split over the blocks of a
 // cluster, every thread owning the same state elements for all tokens, the head's norm summed through distributed shared memory.

@@ -41,8 +41,8 @@ struct FileTensor {
     size_t nbytes = 0;
 };
 
-// The table of a safetensors file: an 8-byte little-endian length, that many bytes of JSON (name -> dtype, shape, data_offsets),
-// then the data.
+// The tensors of a safetensors file.  Layout: u64 header size, a JSON object with one member per tensor, the bytes the members'
+// data_offsets refer to.
 int read_table(const Mapped &f, std::vector<FileTensor> *out) {
     uint64_t len = 0;
     B200_REQUIRE(f.n >= 8, "model_load: the safetensors file is too short");

@@ -95,8 +95,8 @@ def generate(ctx, prompts, max_new, stop=(), max_seqs=16, portion=None):
 
 
 class Replay:
-    """Feeds given tokens step by step and hands out logits (no sampling): the same decode calls, cells and slots the serving
-    loop uses, under the caller's schedule."""
+    """Recorded streams instead of generated ones: tokens and schedule are the caller's, logits come back.  The same decode calls,
+    cells and slots as the serving loop."""
 
     def __init__(self, ctx):
         self.ctx = ctx

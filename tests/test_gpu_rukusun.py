@@ -270,7 +270,7 @@ def test_window_edges_in_prompts_and_decoding(ll, window):
 
 
 def test_window_edges_in_bf16(ll):
-    for window in (64, 72):
+    for window in (64, 81):
         cfg, w = needle(window)
         toks = [t % 59 for t in M.tokens(cfg, 200, 85)]
         toks[40] = 59
