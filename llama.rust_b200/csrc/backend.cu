@@ -1028,7 +1028,7 @@ static int compute_gla(BackendCtx *bc, const ggml_tensor *op) {
     a.a2 = op->src[1]->data; a.a2_type = op->src[1]->type;
     a.a2_bias = (const float *)op->src[2]->data;
     a.norm_w = (const float *)op->src[3]->data;
-    a.state = (float *)op->src[4]->data;
+    a.state = (float *)op->src[4]->data; a.n_slots = op->src[4]->ne[1];
     a.seg = (const int32_t *)op->src[5]->data; a.n_seg = op->src[5]->ne[1];
     a.scratch = op->src[6] ? (float *)op->src[6]->data : nullptr;
     a.y = op->data; a.y_type = op->type; a.ldy = row_ld(op);

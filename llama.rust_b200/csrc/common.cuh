@@ -266,6 +266,12 @@ int launch_rms_norm_w(const float *x, int64_t ldx, const float *w, void *y, int 
 int launch_take_rows(const void *table, int table_type, int64_t ld_table, int64_t table_rows, const int32_t *ids, int64_t n, void *y, int y_type, int64_t ldy,
                      int64_t ne0, float factor, cudaStream_t s);
 
+// One sequence's stretch of a step's rows, as the nodes that follow a sequence read it (I32 [SEG_FIELDS, n_seg]): its first row and
+// rows, its state slot and whether it starts from nothing, the position of its first row, its first entry in the list of cells and
+// the position that entry stands for
+enum { SEG_ROW0 = 0, SEG_ROWS = 1, SEG_SLOT = 2, SEG_FRESH = 3, SEG_POS0 = 4, SEG_TAB0 = 5, SEG_KEY0 = 6, SEG_FIELDS = 8 };
+constexpr int ERR_SEGMENT = 6;   // error code of a kernel that was given a segment outside its rows, slots or segments
+
 // gated linear attention (gla.cu)
 struct GlaArgs {
     const float *proj = nullptr;     // [n][ldp]: q, k, v, g and the decay's low-rank input at the offsets
@@ -275,7 +281,7 @@ struct GlaArgs {
     const float *a2_bias = nullptr, *norm_w = nullptr;
     float *state = nullptr;          // [slot][heads][dim][vdim]
     const int32_t *seg = nullptr;
-    int64_t n_seg = 0;
+    int64_t n_seg = 0, n_slots = 0;
     float *scratch = nullptr;        // null: token by token
     void *y = nullptr;
     int y_type = 0;
@@ -283,6 +289,7 @@ struct GlaArgs {
     int heads = 0, dim = 0, vdim = 0, rank = 0;
     int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a = 0;
     float q_factor = 1.0f, inv_tau = 1.0f, eps = 0.0f;
+    int *err = nullptr;              // set by launch_gla
 };
 size_t gla_scratch_floats(int64_t heads, int64_t dim, int64_t vdim, int64_t n, int64_t n_seg);
 int launch_gla(const GlaArgs &a, cudaStream_t s);

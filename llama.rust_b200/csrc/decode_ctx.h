@@ -38,9 +38,6 @@ struct Weight {
     ggml_backend_buffer_t buf = nullptr;
 };
 
-// One sequence's stretch of a step's rows, as the nodes that follow a sequence read it (I32 [SEG_FIELDS, n_seg] on the device)
-enum { SEG_ROW0 = 0, SEG_ROWS = 1, SEG_SLOT = 2, SEG_FRESH = 3, SEG_POS0 = 4, SEG_TAB0 = 5, SEG_KEY0 = 6, SEG_FIELDS = 8 };
-
 // What a step's graph is built for; equal shapes share one graph
 struct StepShape {
     int64_t n = 0;          // tokens

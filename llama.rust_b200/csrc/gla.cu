@@ -23,15 +23,16 @@ namespace cg = cooperative_groups;
 
 namespace b200 {
 
-// decode_ctx.h's segment fields
-enum { GSEG_ROW0 = 0, GSEG_ROWS = 1, GSEG_SLOT = 2, GSEG_FRESH = 3, GSEG_FIELDS = 8 };
-
 namespace {
 
 constexpr int GLA_THREADS = 256, GLA_SUB = 16;
 
 // log of the decay: log(sigmoid(z)) / tau
 __device__ __forceinline__ float gla_log_decay(float z, float inv_tau) { return -(fmaxf(-z, 0.0f) + log1pf(expf(-fabsf(z)))) * inv_tau; }
+
+__device__ __forceinline__ bool gla_segment_ok(const GlaArgs &a, const int32_t *sg) {
+    return sg[SEG_ROW0] >= 0 && sg[SEG_ROWS] >= 0 && (int64_t)sg[SEG_ROW0] + sg[SEG_ROWS] <= a.n && sg[SEG_SLOT] >= 0 && sg[SEG_SLOT] < a.n_slots;
+}
 
 // ---- token by token ------------------------------------------------------------------------------------------
 template <typename W, typename Y, int VEC>
@@ -46,10 +47,14 @@ gla_step_kernel(GlaArgs a, int lanes, int cols) {
     float *s_a = gla_sm, *s_k = s_a + a.dim, *s_q = s_k + a.dim, *s_red = s_q + a.dim;   // s_red [groups][cols]
     pdl_trigger();
     // the step's inputs are in place before its first kernel starts
-    const int32_t *sg = a.seg + (int64_t)blockIdx.z * GSEG_FIELDS;
-    const int row0 = sg[GSEG_ROW0], rows = sg[GSEG_ROWS];
-    bool fresh = sg[GSEG_FRESH] != 0;
-    float *S = a.state + (((int64_t)sg[GSEG_SLOT] * a.heads + h) * a.dim) * a.vdim + v0;
+    const int32_t *sg = a.seg + (int64_t)blockIdx.z * SEG_FIELDS;
+    const int row0 = sg[SEG_ROW0], rows = sg[SEG_ROWS];
+    if (!gla_segment_ok(a, sg)) {   // (the same for every block of the cluster)
+        if (tid == 0) atomicExch(a.err, ERR_SEGMENT);
+        return;
+    }
+    bool fresh = sg[SEG_FRESH] != 0;
+    float *S = a.state + (((int64_t)sg[SEG_SLOT] * a.heads + h) * a.dim) * a.vdim + v0;
     const W *a2 = (const W *)a.a2 + (int64_t)h * a.dim * a.rank;
     for (int d = tid; d < a.dim; d += GLA_THREADS) {
         for (int c = 0; c < vn; c += 32) l2_prefetch(S + (int64_t)d * a.vdim + c);
@@ -141,15 +146,16 @@ struct GlaScratch {
     float *dC;       // [chunk][head][dim]      the chunk's whole decay
     float *S;        // [chunk][head][dim][vdim] the chunk's contribution, then the state in front of it
     float *o;        // [n][heads][vdim], when a head's values do not fit one block
+    int chunks;      // there is room for
 };
 // chunk ci of the step -> its segment, first row and rows; false past the last
-__device__ __forceinline__ bool gla_find_chunk(const int32_t *seg, int n_seg, int C, int ci, int *row0, int *rows) {
-    for (int s = 0; s < n_seg; s++) {
-        const int n = seg[s * GSEG_FIELDS + GSEG_ROWS], k = (n + C - 1) / C;
+__device__ __forceinline__ bool gla_find_chunk(const GlaArgs &a, int C, int ci, int *row0, int *rows) {
+    for (int s = 0; s < (int)a.n_seg; s++) {
+        const int n = a.seg[s * SEG_FIELDS + SEG_ROWS], k = (n + C - 1) / C;
         if (ci < k) {
-            *row0 = seg[s * GSEG_FIELDS + GSEG_ROW0] + ci * C;
+            *row0 = a.seg[s * SEG_FIELDS + SEG_ROW0] + ci * C;
             *rows = min(C, n - ci * C);
-            return true;
+            return gla_segment_ok(a, a.seg + s * SEG_FIELDS);   // (the scan reports one that is not)
         }
         ci -= k;
     }
@@ -176,7 +182,7 @@ gla_chunk_kernel(GlaArgs a, GlaScratch sc) {
     pdl_trigger();
     pdl_wait();
     int row0, rows;
-    if (!gla_find_chunk(a.seg, (int)a.n_seg, C, ci, &row0, &rows)) return;
+    if (!gla_find_chunk(a, C, ci, &row0, &rows)) return;
     const float *proj = a.proj + (int64_t)row0 * a.ldp;
     const int64_t ch = (int64_t)ci * a.heads + h;
 
@@ -360,7 +366,7 @@ gla_mm_kernel(GlaArgs a, GlaScratch sc, int C) {
     pdl_trigger();
     pdl_wait();
     int row0, rows;
-    if (!gla_find_chunk(a.seg, (int)a.n_seg, C, ci, &row0, &rows)) return;
+    if (!gla_find_chunk(a, C, ci, &row0, &rows)) return;
     const int64_t ch = (int64_t)ci * a.heads + h;
     const float *values = a.proj + (int64_t)row0 * a.ldp + a.off_v + h * a.vdim;
     const int n_state = OUT ? (a.dim + KS - 1) / KS : 0, slabs = n_state + (rows + KS - 1) / KS;
@@ -474,10 +480,14 @@ gla_scan_kernel(GlaArgs a, GlaScratch sc, int C) {
     const int64_t per = (int64_t)a.dim * a.vdim, i = ((int64_t)blockIdx.x * GLA_THREADS + threadIdx.x) * VEC;
     if (i >= per) return;
     int first = 0;
-    for (int s = 0; s < sidx; s++) first += (a.seg[s * GSEG_FIELDS + GSEG_ROWS] + C - 1) / C;
-    const int32_t *sg = a.seg + sidx * GSEG_FIELDS;
-    const int chunks = (sg[GSEG_ROWS] + C - 1) / C, d = (int)(i / a.vdim);
-    float *state = a.state + ((int64_t)sg[GSEG_SLOT] * a.heads + h) * per + i;
+    for (int s = 0; s < sidx; s++) first += (a.seg[s * SEG_FIELDS + SEG_ROWS] + C - 1) / C;
+    const int32_t *sg = a.seg + sidx * SEG_FIELDS;
+    const int chunks = (sg[SEG_ROWS] + C - 1) / C, d = (int)(i / a.vdim);
+    if (!gla_segment_ok(a, sg) || first + chunks > sc.chunks) {
+        if (i == 0) atomicExch(a.err, ERR_SEGMENT);
+        return;
+    }
+    float *state = a.state + ((int64_t)sg[SEG_SLOT] * a.heads + h) * per + i;
     const auto ld = [](const float *p, float (&f)[VEC]) {
         if constexpr (VEC == 4) *reinterpret_cast<float4 *>(f) = *reinterpret_cast<const float4 *>(p);
         else f[0] = *p;
@@ -488,7 +498,7 @@ gla_scan_kernel(GlaArgs a, GlaScratch sc, int C) {
     };
     float s[VEC];
     ld(state, s);
-    if (sg[GSEG_FRESH])
+    if (sg[SEG_FRESH])
 #pragma unroll
         for (int e = 0; e < VEC; e++) s[e] = 0.0f;
     float *p = sc.S + ((int64_t)first * a.heads + h) * per + i;
@@ -567,6 +577,7 @@ int launch_chunks(const GlaArgs &a, cudaStream_t s) {
     GlaScratch sc;
     const unsigned chunks = (unsigned)((a.n + C - 1) / C + a.n_seg);
     const size_t nh = (size_t)chunks * a.heads;
+    sc.chunks = (int)chunks;
     sc.q = a.scratch;
     sc.k = sc.q + round4(nh * C * a.dim);
     sc.A = sc.k + round4(nh * C * a.dim);
@@ -618,7 +629,10 @@ size_t gla_scratch_floats(int64_t heads, int64_t dim, int64_t vdim, int64_t n, i
     return 2 * round4(nh * C * dim) + round4(nh * C * C) + round4(nh * dim) + round4(nh * dim * vdim) + (vdim > 256 ? (size_t)n * heads * vdim : 0);
 }
 
-int launch_gla(const GlaArgs &a, cudaStream_t s) {
+int launch_gla(const GlaArgs &args, cudaStream_t s) {
+    GlaArgs a = args;
+    int rc = device_error_word(&a.err);
+    if (rc != B200_STATUS_SUCCESS) return rc;
     B200_REQUIRE(a.proj && a.a2 && a.a2_bias && a.norm_w && a.state && a.seg && a.y, "gla: null operand");
     B200_REQUIRE(a.heads > 0 && a.dim > 0 && a.vdim > 0 && a.rank > 0 && a.n_seg > 0, "gla: bad shape");
     return a.a2_type == B200_TYPE_F32 ? launch_typed<float>(a, s) : launch_typed<__nv_bfloat16>(a, s);

@@ -16,8 +16,6 @@
 
 namespace b200 {
 
-enum { LSEG_ROW0 = 0, LSEG_ROWS = 1, LSEG_POS0 = 4, LSEG_TAB0 = 5, LSEG_KEY0 = 6, LSEG_FIELDS = 8 };   // decode_ctx.h
-
 namespace {
 
 constexpr int LT = 256;             // threads per block
@@ -168,8 +166,13 @@ latent_decode_kernel(LatentArgs a, int head_groups, int *err) {
     const int pos = a.pos[row];
     const int lo = first_key(a, pos) + split * a.per_split, hi = min(lo + a.per_split, pos + 1);
     if (lo >= hi) return;
-    const int32_t *sg = a.seg + (int64_t)a.row_seg[row] * LSEG_FIELDS;
-    const int tab0 = sg[LSEG_TAB0] - sg[LSEG_KEY0];
+    const int si = a.row_seg[row];
+    if (si < 0 || si >= a.n_seg) {
+        if (tid == 0) atomicExch(err, ERR_SEGMENT);
+        return;
+    }
+    const int32_t *sg = a.seg + (int64_t)si * SEG_FIELDS;
+    const int tab0 = sg[SEG_TAB0] - sg[SEG_KEY0];
     for (int i = tid; i < LH * qs; i += LT) {
         const int h = i / qs, d = i - h * qs;
         sq[i] = h < nh && d < D ? a.queries[(row * a.heads + h0 + h) * D + d] : 0.0f;
@@ -327,14 +330,16 @@ latent_value_kernel(LatentArgs a) {
 
 // ---- many rows ---------------------------------------------------------------------------------------------
 // tile ti of 64 (or `per`) rows -> its segment, first row inside it and rows; false past the last
-__device__ __forceinline__ const int32_t *find_tile(const LatentArgs &a, int per, int ti, int *r0, int *rows) {
+__device__ __forceinline__ const int32_t *find_tile(const LatentArgs &a, int per, int ti, int *r0, int *rows, int *err) {
     for (int s = 0; s < (int)a.n_seg; s++) {
-        const int32_t *sg = a.seg + s * LSEG_FIELDS;
-        const int n = sg[LSEG_ROWS], k = (n + per - 1) / per;
+        const int32_t *sg = a.seg + s * SEG_FIELDS;
+        const int n = sg[SEG_ROWS], k = (n + per - 1) / per;
         if (ti < k) {
             *r0 = ti * per;
             *rows = min(per, n - ti * per);
-            return sg;
+            if (sg[SEG_ROW0] >= 0 && (int64_t)sg[SEG_ROW0] + n <= a.n) return sg;
+            atomicExch(err, ERR_SEGMENT);
+            return nullptr;
         }
         ti -= k;
     }
@@ -350,10 +355,10 @@ latent_attn_kernel(LatentArgs a, int *err) {
     pdl_trigger();
     pdl_wait();
     int r0, rows;
-    const int32_t *sg = find_tile(a, LT / 32, blockIdx.x, &r0, &rows);
+    const int32_t *sg = find_tile(a, LT / 32, blockIdx.x, &r0, &rows, err);
     if (!sg || warp >= rows) return;
-    const int64_t row = sg[LSEG_ROW0] + r0 + warp;
-    const int pos = sg[LSEG_POS0] + r0 + warp, lo = first_key(a, pos);
+    const int64_t row = sg[SEG_ROW0] + r0 + warp;
+    const int pos = sg[SEG_POS0] + r0 + warp, lo = first_key(a, pos);
     if (a.rot_dims > 0 && pos >= a.rope_rows) {
         if (lane == 0) atomicExch(err, ERR_POS);
         return;
@@ -364,7 +369,7 @@ latent_attn_kernel(LatentArgs a, int *err) {
     for (int c = lane; c < a.vdim; c += 32) o[c] = 0.0f;
     __syncwarp();
     float m = -INFINITY, l = 0.0f;
-    const int64_t base = (int64_t)sg[LSEG_TAB0] - sg[LSEG_KEY0];
+    const int64_t base = (int64_t)sg[SEG_TAB0] - sg[SEG_KEY0];
     if (base + lo < 0 || base + pos >= a.n_tab) {
         if (lane == 0) atomicExch(err, ERR_CELL);
         return;
@@ -427,12 +432,12 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
     pdl_wait();
     int r0, rows;
     // later tiles of a prompt see more keys: they go first
-    const int32_t *sg = find_tile(a, MQ, gridDim.x - 1 - blockIdx.x, &r0, &rows);
+    const int32_t *sg = find_tile(a, MQ, gridDim.x - 1 - blockIdx.x, &r0, &rows, err);
     if (!sg) return;
-    const int64_t row0 = sg[LSEG_ROW0] + r0;
-    const int pos0 = sg[LSEG_POS0] + r0, last = pos0 + rows - 1;
+    const int64_t row0 = sg[SEG_ROW0] + r0;
+    const int pos0 = sg[SEG_POS0] + r0, last = pos0 + rows - 1;
     const int lo = first_key(a, pos0);
-    const int64_t base = (int64_t)sg[LSEG_TAB0] - sg[LSEG_KEY0];
+    const int64_t base = (int64_t)sg[SEG_TAB0] - sg[SEG_KEY0];
     if ((a.rot_dims > 0 && last >= a.rope_rows) || base + lo < 0 || base + last >= a.n_tab) {
         if (tid == 0) atomicExch(err, a.rot_dims > 0 && last >= a.rope_rows ? ERR_POS : ERR_CELL);
         return;

@@ -166,3 +166,21 @@ def test_malformed_nodes_are_refused(sess):
     assert not sess.supports(node(sess, LATENT_DECODE, gp.F32, [4, 1, 3], [x, None, w], ints=[(0, 1), (1, 2), (2, 2), (3, 2), (4, 2)]))
     bad = node(sess, DENSE_MM, gp.F32, [9, 3], [w, x])
     assert sess.compute([bad]) != 0 and "dense" in sess.last_error()
+
+
+def test_a_segment_outside_the_step_is_reported(sess):
+    """a slot the state has not, rows the step has not: skipped and reported, the rest of the node unharmed"""
+    H, d, e, R, n = 1, 8, 8, 1, 40
+    rng = np.random.default_rng(1)
+    proj, state = rng.standard_normal((n, 2 * d + 2 * e + R)).astype(np.float32), np.zeros((2, d * e), np.float32)
+    ts = put(sess, state)
+    srcs = [put(sess, proj), put(sess, np.ones((d, R)), gp.BF16), put(sess, np.ones(d)), put(sess, np.ones(e)), ts]
+    for scratch in (None, put(sess, np.zeros(1 << 18, np.float32))):
+        for bad in ([20, 20, 2, 1, 0, 0, 0, 0], [20, 21, 1, 1, 0, 0, 0, 0], [-1, 20, 1, 1, 0, 0, 0, 0]):
+            sess.set(ts, state)
+            y = node(sess, GLA, gp.F32, [H * e, n], srcs + [put(sess, np.array([[0, 20, 0, 1, 0, 0, 0, 0], bad]), gp.I32), scratch],
+                     ints=[(0, H), (1, d), (2, e), (3, 0), (4, d), (5, 2 * d), (6, 2 * d + e), (7, 2 * d + 2 * e), (11, 20), (12, R)], floats=[(8, 1.0), (9, 1.0), (10, 1e-5)])
+            assert sess.compute([y]) == 0, sess.last_error()
+            assert b200.load().kernel_error() == 6
+            after = sess.get(ts, np.float32, 2 * d * e).reshape(2, -1)
+            assert after[0].any() and not after[1].any() and np.isfinite(get(sess, y)[:20]).all()
