@@ -43,14 +43,16 @@ enum {
  * r * n_local; src[1] is a scratch tensor of the node's size. */
 enum { B200_OP_TP_ALL_REDUCE = 0x4200, B200_OP_TP_ALL_GATHER = 0x4201 };
 
-/* Ops outside ggml's enum for decoders with dense weights, recurrent layers and latent attention (arch_rukusun.cpp emits them;
- * every constant is a parameter of the node).  "F32 / BF16" below: rows of either type.  f: the op_params word holds the bits
+/* Ops outside ggml's enum for decoders with dense weights, recurrent layers, latent and grouped-query attention (arch_rukusun.cpp and
+ * arch_lenolix.cpp emit them; every constant is a parameter of the node).  "F32 / BF16" below: rows of either type.  f: the op_params word holds the bits
  * of a float.  A step's sequences: `seg` I32 [8, n_seg] = {first row, rows, state slot, starts from nothing, position of the
- * first row, first entry in tab, position of that entry, -}; `row_seg` I32 [n] the sequence of every row; `tab` I32 [n_tab]
- * the cells of the sequences' positions one after the other; `pos` I32 [n].
+ * first row, first entry in tab, position of the entry after the kept ones, kept entries}; `row_seg` I32 [n] the sequence of every
+ * row; `tab` I32 [n_tab] the cells of the sequences' positions one after the other, the kept first positions ahead; `pos` I32 [n].
  *
- * DENSE_MM       w [k, n] F32 / BF16, x [k, m] F32 / BF16, addend [n, m] F32 or null, norm weight [k] F32 or null -> [n, m] F32 /
- *                BF16: y = act(w (x / rms(x) * norm)) + addend.  op_params: 0 act (0 none, 1 tanh-form gelu), 1 f eps.
+ * DENSE_MM       w [k, n] F32 / BF16, x [k, m] F32 / BF16, addend [n, m] F32 or null, norm weight [k] F32 or null, bias [n] F32 or
+ *                null -> [n, m] F32 / BF16: y = act(w (x / rms(x) * norm) + bias) + addend.  op_params: 0 act (0 none, 1 tanh-form
+ *                gelu, 2 clamped gate: rows 2 i and 2 i + 1 are a gate g and its up row u, min(g, limit) sigmoid(alpha min(g, limit))
+ *                (clamp(u, -limit, limit) + 1), the result [n / 2, m], no addend), 1 f eps, 2 f limit, 3 f alpha.
  * RMS_NORM_W     x F32 rows, weight [ne0] F32 -> F32 / BF16 rows.  op_params: 0 f eps.
  * TAKE_ROWS      table F32 / BF16, ids I32 -> F32 / BF16 rows times a factor.  op_params: 0 f factor.
  * GLA            gated linear attention of every head, its output normed per head and gated: proj F32 [., n] with q, k, v, g and
@@ -68,10 +70,27 @@ enum { B200_OP_TP_ALL_REDUCE = 0x4200, B200_OP_TP_ALL_GATHER = 0x4201 };
  * LATENT_DECODE  queries, pos, cell rows, row_seg, seg, tab -> F32 [rank + 2, heads, splits, n]: per split the weighted sum of
  *                latents, running maximum, sum of weights.
  * LATENT_VALUE   those, pos, ukv, proj, sink [heads] F32 -> F32 / BF16 [heads vdim, n]: splits merged, the value weight, the gate.
- * LATENT_ATTN    proj, pos, kv [heads (dim + vdim), n_tab], latent rows by tab entry, sink, seg -> F32 / BF16 [heads vdim, n]. */
+ * LATENT_ATTN    proj, pos, kv [heads (dim + vdim), n_tab], latent rows by tab entry, sink, seg -> F32 / BF16 [heads vdim, n].
+ * PAIR_EMBED     table, tokens I32 [n], prev I32 [n] (the token before, negative: none), pairs [., buckets + 1] or null, copy F32 / BF16
+ *                [., n] or null -> F32 [., n]: table rows times a factor plus rows (prev mul_prev + token mul_cur) mod buckets of pairs (the
+ *                last row where there is no token before); copy receives the same.  op_params: 0 f factor, 1 mul_prev, 2 mul_cur.
+ * LAYER_NORM_W   x F32 rows, weight [ne0] F32, bias [ne0] F32 or null -> F32 / BF16 rows.  op_params: 0 f eps.
+ * NORM_SUM       x F32 rows, y F32 rows, weight, bias or null, scale or null (F32 [ne0]), next weight or null, next bias or null, next
+ *                rows F32 / BF16 or null -> F32 rows x + layer_norm(y) scale; next rows, if given, receives layer_norm of that with
+ *                the next weight and bias (without a next weight, that itself).  op_params: 0 f eps.
+ * Grouped-query attention, op_params: 0 heads, 1 key heads, 2 dim, 3 vdim, 4 window (0: every earlier position), 5 first positions seen
+ *                whatever their distance, 6 f score factor, 7 rotary dims (channel i turns with i + dims / 2), 8 f rotary base, 9 f
+ *                wavelength factor (0: none), 10 f low, 11 f high, 12 f original length, 13 blocks a row's keys are split over.  proj:
+ *                q of all heads, k, v of all key heads.  A cell's row holds per key head dim key and vdim value channels, each padded to
+ *                a multiple of 8 with zeros.
+ * GROUPED_STORE  proj, pos, cells I32 [n] -> aliases the cell rows it writes.
+ * GROUPED_DECODE proj, pos, cells, cell rows (the rows' own are written), row_seg, seg, tab, sink [heads] F32 or null -> F32 / BF16
+ *                [heads vdim, n].
+ * GROUPED_ATTN   the same operands, the rows' own cells already written. */
 enum { B200_OP_DENSE_MM = 0x4210, B200_OP_RMS_NORM_W = 0x4211, B200_OP_TAKE_ROWS = 0x4212, B200_OP_GLA = 0x4213,
        B200_OP_LATENT_STORE = 0x4214, B200_OP_LATENT_QUERY = 0x4215, B200_OP_LATENT_DECODE = 0x4216, B200_OP_LATENT_VALUE = 0x4217,
-       B200_OP_LATENT_ATTN = 0x4218 };
+       B200_OP_LATENT_ATTN = 0x4218, B200_OP_PAIR_EMBED = 0x4219, B200_OP_LAYER_NORM_W = 0x421a, B200_OP_NORM_SUM = 0x421b,
+       B200_OP_GROUPED_STORE = 0x421c, B200_OP_GROUPED_DECODE = 0x421d, B200_OP_GROUPED_ATTN = 0x421e };
 
 /* enum ggml_unary_op value carried in op_params[0] of a GGML_OP_UNARY node (crates/ggml/src/ops.rs:1632-1636) */
 enum { GGML_UNARY_OP_SILU = 10 };

@@ -7,14 +7,11 @@
 // inside the mat-muls; many rows (BF16 models) hand the mat-muls BF16 rows.  Attention over the latents has two forms as well:
 // queries taken through the key weight, against the cached latents themselves (a few rows per sequence), or keys and values
 // expanded from the latents for the positions the step can see (a prompt's rows).
-#include <cmath>
-
-#include "decode_ctx.h"
+#include "arch_dense.h"
 
 namespace b200 {
 namespace {
 
-constexpr int64_t FEW_ROWS = 16;           // rows up to which activations stay F32 and mat-muls read the weights row by row
 constexpr int64_t GLA_TOKENWISE = 16;      // rows per sequence up to which the recurrence runs token by token
 constexpr int64_t LATENT_FEW = 8;          // rows per sequence up to which attention reads the latents themselves
 constexpr int64_t SPLIT_KEYS = 32;         // keys a split of that attention is cut into
@@ -32,19 +29,13 @@ struct Layer {
     int64_t cell_row() const { return (kv_rank + rot + 7) / 8 * 8; }   // elements of a cell's row
 };
 
-int32_t bits(float f) {
-    int32_t i;
-    memcpy(&i, &f, 4);
-    return i;
-}
-
 class RukusunArch : public Arch {
 public:
     int dtype = B200_TYPE_BF16;
     int64_t vocab = 0, width = 0;
     float eps = 1e-5f, embed_scale = 1.0f;
     std::vector<Layer> layers;
-    int64_t loop_start = 0, loop_stop = 0, loop_times = 0;   // times 0: no loop
+    LoopSpec loop;
 
     const char *name() const override { return "Rukusun"; }
     int32_t n_vocab() const override { return (int32_t)vocab; }
@@ -58,20 +49,7 @@ public:
         }
         return span;
     }
-    // the layers in the order they run: (layer, pass); pass -1 outside the loop
-    std::vector<std::pair<int64_t, int64_t>> runs() const {
-        std::vector<std::pair<int64_t, int64_t>> r;
-        const int64_t n = (int64_t)layers.size();
-        if (loop_times == 0) {
-            for (int64_t i = 0; i < n; i++) r.emplace_back(i, -1);
-            return r;
-        }
-        for (int64_t i = 0; i < loop_start; i++) r.emplace_back(i, -1);
-        for (int64_t t = 0; t < loop_times; t++)
-            for (int64_t i = loop_start; i < loop_stop; i++) r.emplace_back(i, t);
-        for (int64_t i = loop_stop; i < n; i++) r.emplace_back(i, -1);
-        return r;
-    }
+    std::vector<std::pair<int64_t, int64_t>> runs() const { return layer_runs((int64_t)layers.size(), loop); }
 
     // per layer run: the cell rows of a latent-attention layer, the state slots of a linear-attention layer
     int alloc_memory(b200_llama *c) override {
@@ -125,18 +103,11 @@ public:
         };
         if (t == "embed" || t == "head") return matrix(t, width, vocab, 0, vocab);
         if (t == "final.norm") return vec(width, true);
-        if (t == "loop.step" && loop_times > 0) return vec(width, false, loop_times);
-        if (t.size() < 3 || t[0] != 'l') return false;
-        const size_t dot = t.find('.');
-        if (dot == std::string::npos || dot < 2 || dot > 7) return false;
+        if (t == "loop.step" && loop.times > 0) return vec(width, false, loop.times);
         int64_t il = 0;
-        for (size_t i = 1; i < dot; i++) {
-            if (t[i] < '0' || t[i] > '9') return false;
-            il = il * 10 + (t[i] - '0');
-        }
-        if (il >= (int64_t)layers.size()) return false;
+        std::string pre, rest;
+        if (!split_layer_name(t, (int64_t)layers.size(), &il, &pre, &rest)) return false;
         const Layer &l = layers[il];
-        const std::string pre = t.substr(0, dot + 1), rest = t.substr(dot + 1);
         if (rest == "norm1") return vec(width, true);
         if (l.ff > 0) {
             if (rest == "norm2") return vec(width, true);
@@ -169,7 +140,7 @@ public:
     }
     std::vector<std::string> tensor_names() const override {
         std::vector<std::string> v = {"embed", "head", "final.norm"};
-        if (loop_times > 0) v.push_back("loop.step");
+        if (loop.times > 0) v.push_back("loop.step");
         for (size_t i = 0; i < layers.size(); i++) {
             const std::string p = "l" + std::to_string(i) + ".";
             const auto add = [&](std::initializer_list<const char *> names) { for (const char *n : names) v.push_back(p + n); };
@@ -200,35 +171,6 @@ private:
     }
 };
 
-// the nodes of one step
-struct StepBuilder : Builder {
-    int act;      // type of the rows handed to mat-muls
-    bool few;
-    float eps;
-
-    ggml_tensor *dense(ggml_tensor *dst, ggml_tensor *w, ggml_tensor *x, ggml_tensor *addend, ggml_tensor *norm_w, int act_code) {
-        ggml_tensor *t = op(dst, B200_OP_DENSE_MM, w, x, addend, norm_w);
-        t->op_params[0] = act_code;
-        t->op_params[1] = bits(eps);
-        return t;
-    }
-    // w applied to the normed rows: inside the mat-mul while there are few
-    ggml_tensor *normed_dense(ggml_tensor *w, ggml_tensor *x, ggml_tensor *norm_w, int type, int act_code, const char *name) {
-        if (!few) {
-            ggml_tensor *h = op(alloc(act, x->ne[0], x->ne[1]), B200_OP_RMS_NORM_W, x, norm_w);
-            h->op_params[0] = bits(eps);
-            x = h;
-            norm_w = nullptr;
-        }
-        return dense(alloc(type, w->ne[1], x->ne[1], 1, name), w, x, nullptr, norm_w, act_code);
-    }
-    ggml_tensor *take_rows(int type, ggml_tensor *table, ggml_tensor *ids, float factor, ggml_tensor *over_slot, const char *name) {
-        ggml_tensor *t = op(over_slot ? over(over_slot, name) : alloc(type, table->ne[0], ids->ne[0], 1, name), B200_OP_TAKE_ROWS, table, ids);
-        t->op_params[0] = bits(factor);
-        return t;
-    }
-};
-
 int RukusunArch::build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &s) {
     const int64_t n = s.n, E = width;
     StepBuilder b;
@@ -238,22 +180,14 @@ int RukusunArch::build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &
     b.few = n <= FEW_ROWS;
     b.act = dtype == B200_TYPE_F32 || b.few ? B200_TYPE_F32 : B200_TYPE_BF16;
     b.eps = eps;
-    g->tokens = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_tokens");
-    g->pos = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_pos");
-    g->cells = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_cells");
-    g->row_seg = b.alloc(B200_TYPE_I32, n, 1, 1, "inp_row_seg");
-    g->seg = b.alloc(B200_TYPE_I32, SEG_FIELDS, s.n_seg, 1, "inp_seg");
-    g->tab = b.alloc(B200_TYPE_I32, std::max<int64_t>(s.n_tab, 1), 1, 1, "inp_tab");
-    g->out_ids = b.alloc(B200_TYPE_I32, s.n_out, 1, 1, "inp_out_ids");
+    b.inputs(s);
     ggml_tensor *resid[2] = {b.alloc(B200_TYPE_F32, E, n, 1, "resid_a"), b.alloc(B200_TYPE_F32, E, n, 1, "resid_b")};
     int side = 0;
     const auto next_slot = [&]() { return resid[side ^= 1]; };
     const auto W = [&](const std::string &name) { return weight(c, name); };
 
-    for (const std::string &t : tensor_names()) {
-        TensorPlace p;
-        B200_REQUIRE(c->tensors_set.count(t) && place(t, &p) && W(p.dst) != nullptr, "%s: tensor %s has not been set", this->name(), t.c_str());
-    }
+    int rc = require_tensors(c, *this);
+    if (rc != B200_STATUS_SUCCESS) return rc;
 
     ggml_tensor *x = b.take_rows(B200_TYPE_F32, W("embed"), g->tokens, embed_scale, resid[side], "inp_embd");
     const size_t layer_base = b.off;
@@ -262,7 +196,7 @@ int RukusunArch::build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &
         b.off = layer_base;
         const Layer &l = layers[rs[r].first];
         const std::string p = "l" + std::to_string(rs[r].first) + ".";
-        if (rs[r].second >= 0 && rs[r].first == loop_start) {
+        if (rs[r].second >= 0 && rs[r].first == loop.start) {
             ggml_tensor *steps = W("loop.step");
             ggml_tensor *row = b.view_2d(steps, E, 1, steps->nb[1], (size_t)rs[r].second * steps->nb[1]);
             x = b.op(b.over(next_slot(), "loop_step"), GGML_OP_ADD, x, row);
@@ -305,12 +239,7 @@ int RukusunArch::build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &
                 mixed = set(b.op(b.alloc(b.act, l.heads * l.vdim, n, 1, "latent_out"), B200_OP_LATENT_VALUE, part, g->pos, ukv, proj));
                 mixed->src[4] = sink;
             } else {
-                ggml_tensor *st = b.fresh(cache->type, 1);
-                for (int i = 0; i < 4; i++) { st->ne[i] = cache->ne[i]; st->nb[i] = cache->nb[i]; }
-                st->view_src = cache;
-                st->data = cache->data;
-                st->buffer = cache->buffer;
-                set(b.op(st, B200_OP_LATENT_STORE, proj, g->pos, cn, g->cells));
+                set(b.op(b.alias_of(cache), B200_OP_LATENT_STORE, proj, g->pos, cn, g->cells));
                 ggml_tensor *rows = b.take_rows(dtype, cache, g->tab, 1.0f, nullptr, "latent_rows");
                 ggml_tensor *kv = b.dense(b.alloc(dtype, ukv->ne[1], g->tab->ne[0], 1, "latent_kv"), ukv, b.view_2d(rows, R, g->tab->ne[0], rows->nb[1], 0),
                                           nullptr, nullptr, 0);
@@ -334,27 +263,6 @@ int RukusunArch::build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &
     g->bytes = b.high;
     return B200_STATUS_SUCCESS;
 }
-
-// ---- configuration -----------------------------------------------------------------------------------------
-struct Field {
-    std::string *err;
-    const Json *get(const Json &o, const char *key, const char *where) {
-        const Json *v = o.find(key);
-        if (!v && err->empty()) *err = std::string("config: ") + where + " has no '" + key + "'";
-        return v;
-    }
-    double number(const Json &o, const char *key, const char *where) {
-        const Json *v = get(o, key, where);
-        if (!v) return 0.0;
-        if (v->kind != Json::NUM && err->empty()) *err = std::string("config: ") + where + " '" + key + "' is not a number";
-        return v->num;
-    }
-    int64_t size(const Json &o, const char *key, const char *where, int64_t low = 1) {
-        const double v = number(o, key, where);
-        if ((v != std::floor(v) || v < (double)low || v > 1e9) && err->empty()) *err = std::string("config: ") + where + " '" + key + "' is not a usable size";
-        return (int64_t)v;
-    }
-};
 
 }  // namespace
 
@@ -407,13 +315,7 @@ std::unique_ptr<Arch> rukusun_from_config(const Json &config, int dtype, std::st
         }
         a->layers.push_back(l);
     }
-    const Json *loop = config.find("loop");
-    if (loop && !loop->is_null()) {
-        a->loop_start = f.size(*loop, "start", "loop", 0);
-        a->loop_stop = f.size(*loop, "stop", "loop");
-        a->loop_times = f.size(*loop, "times", "loop");
-        if ((a->loop_stop <= a->loop_start || a->loop_stop > (int64_t)a->layers.size()) && err->empty()) *err = "config: the loop's layers are out of range";
-    }
+    a->loop = f.loop(config, (int64_t)a->layers.size());
     if (!err->empty()) return nullptr;
     return a;
 }

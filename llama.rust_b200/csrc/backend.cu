@@ -445,12 +445,14 @@ static bool supports_dense(const ggml_tensor *op, std::string *why) {
     const int32_t *p = op->op_params;
     switch (op->op) {
         case B200_OP_DENSE_MM:
-            if (!dense_rows(a) || !is_contiguous(a) || !dense_rows(b) || !dense_rows(op)) return no("dense mat-mul wants F32 / BF16 rows");
-            if (a->ne[0] != b->ne[0] || op->ne[0] != a->ne[1] || op->ne[1] != b->ne[1]) return no("dense mat-mul: shape");
+            if (!dense_rows(a) || !dense_rows(b) || !dense_rows(op)) return no("dense mat-mul wants F32 / BF16 rows");
+            if (p[0] < ACT_NONE || p[0] > ACT_CLAMPED_GATE) return no("dense mat-mul: activation function");
+            if (p[0] == ACT_CLAMPED_GATE && (a->ne[1] % 2 || op->src[2])) return no("dense mat-mul: a gated result takes pairs of rows and no addend");
+            if (a->ne[0] != b->ne[0] || op->ne[0] != a->ne[1] / (p[0] == ACT_CLAMPED_GATE ? 2 : 1) || op->ne[1] != b->ne[1]) return no("dense mat-mul: shape");
             if (op->src[2] && (!dense_rows(op->src[2]) || op->src[2]->type != B200_TYPE_F32 || op->src[2]->ne[0] != op->ne[0] || op->src[2]->ne[1] != op->ne[1]))
                 return no("dense mat-mul: the addend must be F32 of the result's shape");
             if (op->src[3] && (!f32_vec(op->src[3], a->ne[0]) || b->type != B200_TYPE_F32 || b->ne[1] > DENSE_FEW_ROWS)) return no("dense mat-mul: norm weight");
-            return p[0] == 0 || p[0] == 1 ? true : no("dense mat-mul: activation function");
+            return !op->src[4] || f32_vec(op->src[4], a->ne[1]) ? true : no("dense mat-mul: bias");
         case B200_OP_RMS_NORM_W:
             if (!dense_rows(a) || a->type != B200_TYPE_F32 || !dense_rows(op) || !same_shape(a, op) || !f32_vec(b, a->ne[0])) return no("rms_norm_w wants F32 rows");
             return true;
@@ -469,6 +471,40 @@ static bool supports_dense(const ggml_tensor *op, std::string *why) {
             if (!i32_list(op->src[5], 8) || op->src[5]->ne[0] != 8) return no("gla: segments");
             if (op->src[6] && !f32_vec(op->src[6], (int64_t)gla_scratch_floats(H, d, e, a->ne[1], op->src[5]->ne[1]))) return no("gla: scratch");
             return true;
+        }
+        case B200_OP_LAYER_NORM_W:
+            if (!dense_rows(a) || a->type != B200_TYPE_F32 || !dense_rows(op) || !same_shape(a, op) || !f32_vec(b, a->ne[0]) || (op->src[2] && !f32_vec(op->src[2], a->ne[0])))
+                return no("layer_norm_w wants F32 rows");
+            return true;
+        case B200_OP_NORM_SUM: {
+            const auto vec = [&](const ggml_tensor *t) { return !t || f32_vec(t, op->ne[0]); };
+            const ggml_tensor *h = op->src[7];
+            if (!dense_rows(a) || a->type != B200_TYPE_F32 || !dense_rows(b) || b->type != B200_TYPE_F32 || !dense_rows(op) || op->type != B200_TYPE_F32 || !same_shape(a, op) ||
+                !same_shape(b, op))
+                return no("norm_sum wants F32 rows of one shape");
+            if (!op->src[2] || !vec(op->src[2]) || !vec(op->src[3]) || !vec(op->src[4]) || !vec(op->src[5]) || !vec(op->src[6])) return no("norm_sum: weights");
+            return !h || (dense_rows(h) && same_shape(h, op)) ? true : no("norm_sum: next rows");
+        }
+        case B200_OP_PAIR_EMBED: {
+            const ggml_tensor *prev = op->src[2], *pairs = op->src[3], *copy = op->src[4];
+            if (!dense_rows(a) || !i32_list(b, op->ne[1]) || !dense_rows(op) || op->type != B200_TYPE_F32 || op->ne[0] != a->ne[0]) return no("pair_embed wants F32 / BF16 rows and I32 ids");
+            if (pairs && (!dense_rows(pairs) || pairs->type != a->type || pairs->ne[0] != a->ne[0] || pairs->ne[1] < 2 || p[1] < 0 || p[2] < 0 || !i32_list(prev, op->ne[1])))
+                return no("pair_embed: table of pairs");
+            return !copy || (dense_rows(copy) && same_shape(copy, op)) ? true : no("pair_embed: copy");
+        }
+        case B200_OP_GROUPED_STORE: case B200_OP_GROUPED_DECODE: case B200_OP_GROUPED_ATTN: {
+            const int64_t H = p[0], G = p[1], d = p[2], e = p[3];
+            if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || p[4] < 0 || p[5] < 0 || p[7] < 0 || p[7] % 2 || p[7] > d) return no("grouped attention: parameters");
+            if (!dense_rows(a) || a->type != B200_TYPE_F32 || a->ne[0] < (H + G) * d + G * e) return no("grouped attention: projection rows");
+            const int64_t n = a->ne[1];
+            const ggml_tensor *cache = op->op == B200_OP_GROUPED_STORE ? op : op->src[3];
+            if (!i32_list(b, n) || !i32_list(op->src[2], n)) return no("grouped attention: positions and cells");
+            if (!dense_rows(cache) || cache->ne[0] < G * (grouped_pad(d) + grouped_pad(e)) || cache->nb[1] % 16) return no("grouped attention: cell rows");
+            if (op->op == B200_OP_GROUPED_STORE) return true;
+            if (!i32_list(op->src[4], n) || !i32_list(op->src[5], SEG_FIELDS) || op->src[5]->ne[0] != SEG_FIELDS || !i32_list(op->src[6], 1)) return no("grouped attention: segments");
+            if (op->src[7] && !f32_vec(op->src[7], H)) return no("grouped attention: sinks");
+            if (op->op == B200_OP_GROUPED_DECODE && (p[13] < 1 || p[13] > 8 || (p[13] & (p[13] - 1)))) return no("grouped attention: splits");
+            return dense_rows(op) && op->ne[0] == H * e && op->ne[1] == n ? true : no("grouped attention: result");
         }
         default: break;
     }
@@ -507,7 +543,8 @@ static bool supports_dense(const ggml_tensor *op, std::string *why) {
 static bool op_supported(const ggml_tensor *op, std::string *why) {
     switch (op->op) {
         case B200_OP_DENSE_MM: case B200_OP_RMS_NORM_W: case B200_OP_TAKE_ROWS: case B200_OP_GLA: case B200_OP_LATENT_STORE: case B200_OP_LATENT_QUERY:
-        case B200_OP_LATENT_DECODE: case B200_OP_LATENT_VALUE: case B200_OP_LATENT_ATTN:
+        case B200_OP_LATENT_DECODE: case B200_OP_LATENT_VALUE: case B200_OP_LATENT_ATTN: case B200_OP_PAIR_EMBED: case B200_OP_LAYER_NORM_W:
+        case B200_OP_NORM_SUM: case B200_OP_GROUPED_STORE: case B200_OP_GROUPED_DECODE: case B200_OP_GROUPED_ATTN:
             return supports_dense(op, why);
         case B200_OP_TP_ALL_REDUCE: case B200_OP_TP_ALL_GATHER: return supports_tp(op, why);
         case GGML_OP_NONE: case GGML_OP_RESHAPE: case GGML_OP_VIEW: case GGML_OP_PERMUTE: case GGML_OP_TRANSPOSE:
@@ -970,12 +1007,49 @@ static int compute_rope(BackendCtx *bc, const ggml_tensor *op) {
 }
 
 // ---- ops of decoders with dense weights --------------------------------------------------------------------
-// Rotary (cos, sin) pairs of a latent-attention node's positions: angles in double precision, position * base^(-2 i / dims)
-static std::vector<int32_t> latent_rope_key(const ggml_tensor *op) { return {0x4c61744e, op->op_params[8], op->op_params[9]}; }
-static bool latent_rotates(const ggml_tensor *op) {
-    return (op->op == B200_OP_LATENT_STORE || op->op == B200_OP_LATENT_QUERY || op->op == B200_OP_LATENT_ATTN) && op->op_params[9] > 0;
+// Rotary (cos, sin) pairs of the attention nodes' positions: angles in double precision, position times a frequency per pair,
+// base^(-2 i / dims).  With a wavelength factor, waves longer than original / low are stretched by it, those shorter than original /
+// high kept, the ones between on a ramp in original / wavelength.
+struct AttnRope {
+    int dims = 0;
+    float base = 0.0f, factor = 0.0f, low = 0.0f, high = 0.0f, original = 0.0f;
+    std::vector<int32_t> key() const {
+        std::vector<int32_t> k = {0x4c61744e, 0, dims, 0, 0, 0, 0};
+        memcpy(&k[1], &base, 4);
+        memcpy(&k[3], &factor, 4);
+        memcpy(&k[4], &low, 4);
+        memcpy(&k[5], &high, 4);
+        memcpy(&k[6], &original, 4);
+        return k;
+    }
+    double frequency(int i) const {
+        const double f = pow((double)base, -2.0 * i / dims);
+        if (factor == 0.0f) return f;
+        const double wave = 2.0 * 3.14159265358979323846 / f;
+        if (wave < (double)original / high) return f;
+        if (wave > (double)original / low) return f / factor;
+        const double keep = ((double)original / wave - low) / ((double)high - low);
+        return (1.0 - keep) * f / factor + keep * f;
+    }
+};
+static AttnRope attn_rope(const ggml_tensor *op) {
+    AttnRope r;
+    if (op->op == B200_OP_LATENT_STORE || op->op == B200_OP_LATENT_QUERY || op->op == B200_OP_LATENT_ATTN) {
+        r.dims = op->op_params[9];
+        r.base = param_f32(op, 8);
+    } else if (op->op == B200_OP_GROUPED_STORE || op->op == B200_OP_GROUPED_DECODE || op->op == B200_OP_GROUPED_ATTN) {
+        r.dims = op->op_params[7];
+        r.base = param_f32(op, 8);
+        r.factor = param_f32(op, 9);
+        if (r.factor != 0.0f) {
+            r.low = param_f32(op, 10);
+            r.high = param_f32(op, 11);
+            r.original = param_f32(op, 12);
+        }
+    }
+    return r;
 }
-static int latent_rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
+static int attn_rope_prepare(BackendCtx *bc, const ggml_tensor *op, const AttnRope &r) {
     const ggml_tensor *pos = op->src[1];
     std::vector<int32_t> p;
     if (in_our_buffer(pos)) {
@@ -991,33 +1065,44 @@ static int latent_rope_prepare(BackendCtx *bc, const ggml_tensor *op) {
         B200_CUDA(cudaMemcpy(p.data(), pos->data, p.size() * 4, cudaMemcpyDeviceToHost));
     }
     const int32_t pmin = *std::min_element(p.begin(), p.end()), pmax = *std::max_element(p.begin(), p.end());
-    B200_REQUIRE(pmin >= 0 && pmax < ROPE_TABLE_MAX_ROWS, "latent attention: position %d out of range", pmin < 0 ? pmin : pmax);
-    const int dims = op->op_params[9];
-    const double base = (double)param_f32(op, 8);
-    return rope_reserve(bc, latent_rope_key(op), pmax, [&](const std::vector<int32_t> &all) {
-        bc->rope_host.resize(all.size() * (size_t)dims);
-        for (int i = 0; i < dims / 2; i++) {
-            const double f = pow(base, -2.0 * i / dims);
-            for (size_t r = 0; r < all.size(); r++) {
-                bc->rope_host[r * dims + 2 * i] = (float)cos((double)all[r] * f);
-                bc->rope_host[r * dims + 2 * i + 1] = (float)sin((double)all[r] * f);
+    B200_REQUIRE(pmin >= 0 && pmax < ROPE_TABLE_MAX_ROWS, "attention: position %d out of range", pmin < 0 ? pmin : pmax);
+    return rope_reserve(bc, r.key(), pmax, [&](const std::vector<int32_t> &all) {
+        bc->rope_host.resize(all.size() * (size_t)r.dims);
+        for (int i = 0; i < r.dims / 2; i++) {
+            const double f = r.frequency(i);
+            for (size_t row = 0; row < all.size(); row++) {
+                bc->rope_host[row * r.dims + 2 * i] = (float)cos((double)all[row] * f);
+                bc->rope_host[row * r.dims + 2 * i + 1] = (float)sin((double)all[row] * f);
             }
         }
         return (int)B200_STATUS_SUCCESS;
     });
 }
+static int attn_rope_table(BackendCtx *bc, const AttnRope &r, const float **table, int64_t *rows) {
+    if (r.dims == 0) return B200_STATUS_SUCCESS;
+    const std::vector<int32_t> key = r.key();
+    for (auto &t : bc->rope_by_pos)
+        if (t.key == key && t.dev) {
+            *table = t.dev;
+            *rows = t.rows;
+            return B200_STATUS_SUCCESS;
+        }
+    B200_REQUIRE(false, "attention: no rotary table");
+}
 
 static int compute_dense_mm(BackendCtx *bc, const ggml_tensor *op) {
     const ggml_tensor *w = op->src[0], *x = op->src[1], *add = op->src[2], *nw = op->src[3];
     DenseMm d;
-    d.w = w->data; d.w_type = w->type;
+    d.w = w->data; d.w_type = w->type; d.ldw = row_ld(w);
     d.x = x->data; d.x_type = x->type; d.ldx = row_ld(x);
     d.y = op->data; d.y_type = op->type; d.ldy = row_ld(op);
     d.addend = add ? (const float *)add->data : nullptr;
     d.ld_addend = add ? row_ld(add) : 0;
     d.norm_w = nw ? (const float *)nw->data : nullptr;
+    d.bias = op->src[4] ? (const float *)op->src[4]->data : nullptr;
     d.act = op->op_params[0];
     d.eps = param_f32(op, 1);
+    d.act_limit = param_f32(op, 2); d.act_alpha = param_f32(op, 3);
     d.n = w->ne[1]; d.k = w->ne[0]; d.m = x->ne[1];
     return launch_dense_mm(d, bc->stream);
 }
@@ -1045,11 +1130,9 @@ static int compute_latent(BackendCtx *bc, const ggml_tensor *op) {
     a.off_q = p[10]; a.off_c = p[11]; a.off_g = p[12];
     a.per_split = p[13]; a.n_splits = p[14];
     a.pos = (const int32_t *)op->src[1]->data;
-    if (latent_rotates(op)) {
-        const std::vector<int32_t> key = latent_rope_key(op);
-        for (auto &t : bc->rope_by_pos)
-            if (t.key == key && t.dev) { a.rope = t.dev; a.rope_rows = t.rows; }
-        B200_REQUIRE(a.rope != nullptr, "latent attention: no rotary table");
+    {
+        int rc = attn_rope_table(bc, attn_rope(op), &a.rope, &a.rope_rows);
+        if (rc != B200_STATUS_SUCCESS) return rc;
     }
     const auto proj = [&](const ggml_tensor *t) { a.proj = (const float *)t->data; a.ldp = row_ld(t); a.n = t->ne[1]; };
     const auto cells = [&](const ggml_tensor *t) { a.cache = t->data; a.ldc = row_ld(t); a.n_cells = t->ne[1]; a.type = t->type; };
@@ -1095,6 +1178,63 @@ static int compute_latent(BackendCtx *bc, const ggml_tensor *op) {
             result();
             return launch_latent_attn(a, bc->stream);
     }
+}
+
+static const float *f32_data(const ggml_tensor *t) { return t ? (const float *)t->data : nullptr; }
+static int compute_layer_norm(BackendCtx *bc, const ggml_tensor *op) {
+    NormSum a;
+    a.x = f32_data(op->src[0]); a.ldx = row_ld(op->src[0]);
+    a.w2 = f32_data(op->src[1]); a.b2 = f32_data(op->src[2]);
+    a.h = op->data; a.h_type = op->type; a.ldh = row_ld(op);
+    a.ne0 = op->ne[0]; a.n = op->ne[1]; a.eps = param_f32(op, 0);
+    return launch_norm_sum(a, bc->stream);
+}
+static int compute_norm_sum(BackendCtx *bc, const ggml_tensor *op) {
+    NormSum a;
+    a.x = f32_data(op->src[0]); a.ldx = row_ld(op->src[0]);
+    a.y = f32_data(op->src[1]); a.ldy = row_ld(op->src[1]);
+    a.w1 = f32_data(op->src[2]); a.b1 = f32_data(op->src[3]); a.scale = f32_data(op->src[4]);
+    a.sum = (float *)op->data; a.ld_sum = row_ld(op);
+    a.w2 = f32_data(op->src[5]); a.b2 = f32_data(op->src[6]);
+    if (op->src[7]) { a.h = op->src[7]->data; a.h_type = op->src[7]->type; a.ldh = row_ld(op->src[7]); }
+    a.ne0 = op->ne[0]; a.n = op->ne[1]; a.eps = param_f32(op, 0);
+    return launch_norm_sum(a, bc->stream);
+}
+static int compute_pair_embed(BackendCtx *bc, const ggml_tensor *op) {
+    const ggml_tensor *t = op->src[0], *pairs = op->src[3], *copy = op->src[4];
+    PairEmbed a;
+    a.table = t->data; a.type = t->type; a.table_rows = t->ne[1]; a.ld_table = row_ld(t);
+    a.tokens = (const int32_t *)op->src[1]->data;
+    if (pairs) {
+        a.pairs = pairs->data; a.ld_pairs = row_ld(pairs); a.buckets = pairs->ne[1] - 1;
+        a.prev = (const int32_t *)op->src[2]->data;
+    }
+    a.factor = param_f32(op, 0); a.mul_prev = op->op_params[1]; a.mul_cur = op->op_params[2];
+    a.y = (float *)op->data; a.ldy = row_ld(op);
+    if (copy) { a.h = copy->data; a.h_type = copy->type; a.ldh = row_ld(copy); }
+    a.ne0 = op->ne[0]; a.n = op->ne[1];
+    return launch_pair_embed(a, bc->stream);
+}
+static int compute_grouped(BackendCtx *bc, const ggml_tensor *op) {
+    const int32_t *p = op->op_params;
+    const bool store = op->op == B200_OP_GROUPED_STORE;
+    const ggml_tensor *proj = op->src[0], *cache = store ? op : op->src[3];
+    GroupedArgs a;
+    a.heads = p[0]; a.kv_heads = p[1]; a.dim = p[2]; a.vdim = p[3]; a.window = p[4]; a.keep = p[5]; a.rot_dims = p[7]; a.splits = p[13];
+    a.scale = param_f32(op, 6);
+    a.proj = f32_data(proj); a.ldp = row_ld(proj); a.n = proj->ne[1];
+    a.pos = (const int32_t *)op->src[1]->data;
+    a.cells = (const int32_t *)op->src[2]->data;
+    a.cache = cache->data; a.type = cache->type; a.ldc = row_ld(cache); a.n_cells = cache->ne[1];
+    int rc = attn_rope_table(bc, attn_rope(op), &a.rope, &a.rope_rows);
+    if (rc != B200_STATUS_SUCCESS) return rc;
+    if (store) return launch_grouped_store(a, bc->stream);
+    a.row_seg = (const int32_t *)op->src[4]->data;
+    a.seg = (const int32_t *)op->src[5]->data; a.n_seg = op->src[5]->ne[1];
+    a.tab = (const int32_t *)op->src[6]->data; a.n_tab = op->src[6]->ne[0];
+    a.sink = f32_data(op->src[7]);
+    a.y = op->data; a.y_type = op->type; a.ldy = row_ld(op);
+    return op->op == B200_OP_GROUPED_DECODE ? launch_grouped_decode(a, bc->stream) : launch_grouped_attn(a, bc->stream);
 }
 
 static int compute_set_rows(BackendCtx *bc, const ggml_tensor *op) {
@@ -1810,6 +1950,10 @@ static int run_nodes(BackendCtx *bc, ggml_cgraph *g) {
             case B200_OP_LATENT_STORE: case B200_OP_LATENT_QUERY: case B200_OP_LATENT_DECODE: case B200_OP_LATENT_VALUE: case B200_OP_LATENT_ATTN:
                 rc = compute_latent(bc, op);
                 break;
+            case B200_OP_PAIR_EMBED: rc = compute_pair_embed(bc, op); break;
+            case B200_OP_LAYER_NORM_W: rc = compute_layer_norm(bc, op); break;
+            case B200_OP_NORM_SUM: rc = compute_norm_sum(bc, op); break;
+            case B200_OP_GROUPED_STORE: case B200_OP_GROUPED_DECODE: case B200_OP_GROUPED_ATTN: rc = compute_grouped(bc, op); break;
             case B200_OP_TP_ALL_REDUCE:
                 rc = tp_all_reduce(bc->tp, (float *)op->data, (int64_t)(ggml_nbytes(op) / 4), bc->stream, &bc->capturable);
                 break;
@@ -1891,8 +2035,9 @@ static int backend_graph_compute(ggml_backend_t be, ggml_cgraph *g) {
             int rc = rope_prepare(bc, op);
             if (rc != B200_STATUS_SUCCESS) return rc;
         }
-        if (op && latent_rotates(op) && supports_dense(op, nullptr)) {
-            int rc = latent_rope_prepare(bc, op);
+        const AttnRope turn = op ? attn_rope(op) : AttnRope();
+        if (turn.dims > 0 && supports_dense(op, nullptr)) {
+            int rc = attn_rope_prepare(bc, op, turn);
             if (rc != B200_STATUS_SUCCESS) return rc;
         }
         if (op && (op->op == B200_OP_TP_ALL_REDUCE || op->op == B200_OP_TP_ALL_GATHER)) {

@@ -239,15 +239,18 @@ int launch_get_rows(int type, const void *table, int64_t ne0, int64_t table_rows
                     int64_t out_stride, cudaStream_t s);
 int launch_argmax(const float *x, int64_t x_stride, int64_t ne0, int64_t nrows, int32_t *out, cudaStream_t s);
 
-// dense mat-muls (dense_mm.cu): y[m][n] = act(w x') + addend with w [n][k] F32 or BF16 rows, x [m][k] F32 or BF16 rows and, with
-// norm_w, x' = x / rms(x) * norm_w (few rows only)
+// dense mat-muls (dense_mm.cu): y[m][n] = act(w x' + bias) + addend with w [n][k] F32 or BF16 rows, x [m][k] F32 or BF16 rows and,
+// with norm_w, x' = x / rms(x) * norm_w (few rows only).  A gated act takes the rows 2 i (gate) and 2 i + 1 (up) together: y is [m][n / 2]
+// ACT_CLAMPED_GATE: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1)
+enum { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_CLAMPED_GATE = 2 };
 constexpr int DENSE_FEW_ROWS = 16;   // activation rows up to which the weights are read row by row
 struct DenseMm {
     const void *w = nullptr;
     int w_type = 0;
+    int64_t ldw = 0;                 // elements, as the other row strides
     const void *x = nullptr;
     int x_type = 0;
-    int64_t ldx = 0;                 // elements
+    int64_t ldx = 0;
     void *y = nullptr;
     int y_type = 0;
     int64_t ldy = 0;
@@ -255,7 +258,9 @@ struct DenseMm {
     int64_t ld_addend = 0;
     const float *norm_w = nullptr;
     float eps = 0.0f;
-    int act = 0;                     // 0: none, 1: tanh-form gelu
+    const float *bias = nullptr;     // [n]
+    int act = ACT_NONE;
+    float act_limit = 0.0f, act_alpha = 0.0f;   // of the gated act
     int64_t n = 0, k = 0, m = 0;
 };
 int launch_dense_mm(const DenseMm &d, cudaStream_t s);
@@ -266,10 +271,46 @@ int launch_rms_norm_w(const float *x, int64_t ldx, const float *w, void *y, int 
 int launch_take_rows(const void *table, int table_type, int64_t ld_table, int64_t table_rows, const int32_t *ids, int64_t n, void *y, int y_type, int64_t ldy,
                      int64_t ne0, float factor, cudaStream_t s);
 
+// layer norms around a residual sum (norm_sum.cu): x' = x + norm(y) scale, then h = norm(x').  norm(v) = (v - mean) / sqrt(variance +
+// eps) w + b.  y null: x' = x (nothing stored); w2 null: h is x' itself; h null: no second result.
+struct NormSum {
+    const float *x = nullptr;
+    int64_t ldx = 0;
+    const float *y = nullptr;
+    int64_t ldy = 0;
+    const float *w1 = nullptr, *b1 = nullptr, *scale = nullptr;   // b1, scale: may be null
+    float *sum = nullptr;                                         // x', may be x
+    int64_t ld_sum = 0;
+    const float *w2 = nullptr, *b2 = nullptr;
+    void *h = nullptr;
+    int h_type = 0;
+    int64_t ldh = 0;
+    int64_t ne0 = 0, n = 0;
+    float eps = 0.0f;
+};
+int launch_norm_sum(const NormSum &a, cudaStream_t s);
+// token embeddings times a factor plus rows of a table of token pairs: row (prev mul_prev + token mul_cur) mod buckets, row `buckets`
+// where prev is negative (norm_sum.cu)
+struct PairEmbed {
+    const void *table = nullptr, *pairs = nullptr;   // of one type; pairs may be null
+    int type = 0;
+    int64_t table_rows = 0, ld_table = 0, ld_pairs = 0;
+    const int32_t *tokens = nullptr, *prev = nullptr;
+    int64_t buckets = 0, mul_prev = 0, mul_cur = 0;
+    float factor = 1.0f;
+    float *y = nullptr;
+    int64_t ldy = 0;
+    void *h = nullptr;                               // a second copy, may be null
+    int h_type = 0;
+    int64_t ldh = 0;
+    int64_t ne0 = 0, n = 0;
+};
+int launch_pair_embed(const PairEmbed &a, cudaStream_t s);
+
 // One sequence's stretch of a step's rows, as the nodes that follow a sequence read it (I32 [SEG_FIELDS, n_seg]): its first row and
-// rows, its state slot and whether it starts from nothing, the position of its first row, its first entry in the list of cells and
-// the position that entry stands for
-enum { SEG_ROW0 = 0, SEG_ROWS = 1, SEG_SLOT = 2, SEG_FRESH = 3, SEG_POS0 = 4, SEG_TAB0 = 5, SEG_KEY0 = 6, SEG_FIELDS = 8 };
+// rows, its state slot and whether it starts from nothing, the position of its first row, its first entry in the list of cells, how
+// many of the entries from there are those of positions 0, 1, .. (kept for good), and the position the entry after them stands for
+enum { SEG_ROW0 = 0, SEG_ROWS = 1, SEG_SLOT = 2, SEG_FRESH = 3, SEG_POS0 = 4, SEG_TAB0 = 5, SEG_KEY0 = 6, SEG_KEPT = 7, SEG_FIELDS = 8 };
 constexpr int ERR_SEGMENT = 6;   // error code of a kernel that was given a segment outside its rows, slots or segments
 
 // gated linear attention (gla.cu)
@@ -328,6 +369,33 @@ int launch_latent_query(const LatentArgs &a, cudaStream_t s);
 int launch_latent_decode(const LatentArgs &a, cudaStream_t s);
 int launch_latent_value(const LatentArgs &a, cudaStream_t s);
 int launch_latent_attn(const LatentArgs &a, cudaStream_t s);   // cache: the rows by tab entry (ldc apart)
+
+// grouped-query attention with a window, kept first tokens and a sink (grouped_attn.cu)
+struct GroupedArgs {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, window = 0, keep = 0, rot_dims = 0;   // window 0: every earlier position
+    float scale = 1.0f;
+    int splits = 1;                  // blocks a (row, key head) of the few-rows kernel is cut into
+    int64_t n = 0;
+    const float *proj = nullptr;     // [n][ldp]: q of all heads, k, v of all key heads
+    int64_t ldp = 0;
+    const int32_t *pos = nullptr;
+    const float *rope = nullptr;     // [rope_rows][rot_dims]: (cos, sin) pairs by position
+    int64_t rope_rows = 0;
+    const int32_t *cells = nullptr;  // the cell each row is stored in
+    void *cache = nullptr;           // [n_cells][ldc]: per key head grouped_pad(dim) key channels, grouped_pad(vdim) value channels
+    int type = 0;
+    int64_t ldc = 0, n_cells = 0;
+    const int32_t *row_seg = nullptr, *seg = nullptr, *tab = nullptr;
+    int64_t n_seg = 0, n_tab = 0;
+    const float *sink = nullptr;     // [heads], may be null
+    void *y = nullptr;
+    int y_type = 0;
+    int64_t ldy = 0;
+};
+inline int64_t grouped_pad(int64_t channels) { return (channels + 7) / 8 * 8; }
+int launch_grouped_store(const GroupedArgs &a, cudaStream_t s);
+int launch_grouped_decode(const GroupedArgs &a, cudaStream_t s);   // stores the rows' own cells too
+int launch_grouped_attn(const GroupedArgs &a, cudaStream_t s);     // their cells have been stored
 
 // scratch owned by the library (one growing allocation per device)
 int scratch_get(size_t bytes, void **ptr);

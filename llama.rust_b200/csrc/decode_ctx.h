@@ -57,15 +57,16 @@ struct Graph {
     std::vector<ggml_tensor *> nodes;
     ggml_tensor *tokens = nullptr, *pos = nullptr, *mask = nullptr, *row_idx = nullptr, *out_ids = nullptr;
     ggml_tensor *seg = nullptr, *row_seg = nullptr, *cells = nullptr, *tab = nullptr;
+    ggml_tensor *prev = nullptr;          // the token before each token in its sequence, -1 for the first (null: not wanted)
     ggml_tensor *logits = nullptr, *argmax = nullptr;
     size_t bytes = 0;                     // compute-buffer bytes the graph spans
 };
 
-// Where a tensor of the model's files goes: rows row0 .. of the device tensor `dst` ([ne0, ne1] of `type`)
+// Where a tensor of the model's files goes: rows row0, row0 + row_step, .. of the device tensor `dst` ([ne0, ne1] of `type`)
 struct TensorPlace {
     std::string dst;
     int type = 0;
-    int64_t ne0 = 0, ne1 = 0, row0 = 0, rows = 0;
+    int64_t ne0 = 0, ne1 = 0, row0 = 0, rows = 0, row_step = 1;
     bool plus_one = false;   // the file holds the distance from one
 };
 
@@ -82,6 +83,8 @@ public:
     // segmented architectures: how many positions back any layer looks, the token itself included (0: everything; -1: no
     // layer keeps keys).  Cells further back are given back as the sequence grows.
     virtual int64_t key_span() const { return 0; }
+    // with a key_span above 0: how many of a sequence's first positions every later token may see all the same.  Their cells stay.
+    virtual int64_t kept_first() const { return 0; }
     virtual int alloc_memory(b200_llama *c) = 0;
     virtual int build(b200_llama *c, Graph *g, uint8_t *base, const StepShape &shape) = 0;
     // the shapes the compute buffer has to hold
@@ -96,13 +99,15 @@ std::unique_ptr<Arch> make_llama_arch(const b200_llama_hparams &hp);
 // nullptr and *err when the configuration does not describe a model of the architecture; dtype: B200_TYPE_BF16 / B200_TYPE_F32
 typedef std::unique_ptr<Arch> (*ArchFromConfig)(const Json &config, int dtype, std::string *err);
 std::unique_ptr<Arch> rukusun_from_config(const Json &config, int dtype, std::string *err);
+std::unique_ptr<Arch> lenolix_from_config(const Json &config, int dtype, std::string *err);
 
-// A sequence of a segmented architecture: the cells of its positions (those before `kept` have been given back), its next
-// position and its state slot.
+// A sequence of a segmented architecture: the cells of the first positions it keeps for good, those of its positions from `kept` on
+// (what stands between has been given back), its next position, its last token and its state slot.
 struct Sequence {
-    std::vector<int32_t> cells;
+    std::vector<int32_t> first_cells, cells;
     int64_t kept = 0;
     int64_t next_pos = 0;
+    int32_t last_token = -1;
     int32_t slot = -1;
 };
 
@@ -133,7 +138,7 @@ struct b200_llama {
     b200::Graph *last = nullptr;
     std::vector<uint16_t> mask_host;
     std::vector<int64_t> idx_host;
-    std::vector<int32_t> seg_host, row_seg_host, cells_host, tab_host;
+    std::vector<int32_t> seg_host, row_seg_host, cells_host, tab_host, prev_host;
     // tensor parallel: this rank holds n_head / tp_size heads, n_head_kv / tp_size cache heads, the matching
     // rows / columns of every matrix (tp.cpp) and 1 / tp_size of the vocabulary rows
     int32_t tp_rank = 0, tp_size = 1;

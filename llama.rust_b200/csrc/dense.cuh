@@ -51,6 +51,11 @@ __device__ __forceinline__ float block_sum(float v, float *part) {
 __device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float dense_act(int act, float v) { return act == 1 ? gelu_tanh(v) : v; }
+__device__ __forceinline__ float dense_act(int act, float v) { return act == ACT_GELU_TANH ? gelu_tanh(v) : v; }
+__device__ __forceinline__ float clamped_gate(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
 
 }  // namespace b200

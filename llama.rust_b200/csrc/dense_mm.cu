@@ -45,7 +45,7 @@ dense_rows_kernel(DenseMm d, int m0, int wpr) {
     const int64_t k = d.k;
     const W *w[RPW];
 #pragma unroll
-    for (int r = 0; r < RPW; r++) w[r] = (const W *)d.w + (row0 + r < d.n ? row0 + r : d.n - 1) * k;
+    for (int r = 0; r < RPW; r++) w[r] = (const W *)d.w + (row0 + r < d.n ? row0 + r : d.n - 1) * d.ldw;
     const float *x = (const float *)d.x + (int64_t)m0 * d.ldx;
     const int64_t step = (int64_t)32 * E * wpr;
     int64_t i = ((int64_t)sub * 32 + lane) * E;
@@ -137,15 +137,29 @@ dense_rows_kernel(DenseMm d, int m0, int wpr) {
     else __syncwarp();
     if (sub != 0 || lane >= RPW * NCOL) return;
     const int r = lane / NCOL, c = lane % NCOL;
-    float v = 0.0f, s = 0.0f;
+    const bool gated = d.act == ACT_CLAMPED_GATE;
+    float v = 0.0f, v2 = 0.0f, s = 0.0f;
     for (int p = 0; p < wpr; p++) {
         v += part[warp + p][r * NCOL + c];
+        if (gated && !(r & 1)) v2 += part[warp + p][(r + 1) * NCOL + c];
         s += part[warp + p][RPW * NCOL + c];
     }
-    const int64_t row = row0 + r, col = m0 + c;
-    if (row >= d.n) return;
-    if (d.norm_w) v *= 1.0f / sqrtf(s / (float)k + d.eps);
-    v = dense_act(d.act, v);
+    int64_t row = row0 + r;
+    const int64_t col = m0 + c;
+    if (row >= d.n || (gated && (r & 1))) return;
+    if (d.norm_w) {
+        const float f = 1.0f / sqrtf(s / (float)k + d.eps);
+        v *= f;
+        v2 *= f;
+    }
+    if (d.bias) v += d.bias[row];
+    if (gated) {
+        if (d.bias) v2 += d.bias[row + 1];
+        v = clamped_gate(v, v2, d.act_limit, d.act_alpha);
+        row >>= 1;
+    } else {
+        v = dense_act(d.act, v);
+    }
     if (d.addend) v += d.addend[col * d.ld_addend + row];
     if (d.y_type == B200_TYPE_F32) ((float *)d.y)[col * d.ldy + row] = v;
     else ((__nv_bfloat16 *)d.y)[col * d.ldy + row] = __float2bfloat16_rn(v);
@@ -167,7 +181,7 @@ template <typename W>
 int launch_few(const DenseMm &d, cudaStream_t s) {
     int dev = 0, sms = 148;
     if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
-    const bool vec = d.k % WLoad<W>::E == 0 && d.k % 4 == 0 && d.ldx % 4 == 0 && (((uintptr_t)d.w | (uintptr_t)d.x | (uintptr_t)d.norm_w) & 15) == 0;
+    const bool vec = d.k % WLoad<W>::E == 0 && d.ldw % WLoad<W>::E == 0 && d.k % 4 == 0 && d.ldx % 4 == 0 && (((uintptr_t)d.w | (uintptr_t)d.x | (uintptr_t)d.norm_w) & 15) == 0;
     int rc = B200_STATUS_SUCCESS;
     for (int64_t m0 = 0; m0 < d.m && rc == B200_STATUS_SUCCESS;) {
         const int64_t left = d.m - m0;
@@ -193,7 +207,7 @@ dense_tiled_kernel(DenseMm d) {
         for (int i = threadIdx.x; i < DT * DTK; i += 256) {
             const int r = i / DTK, kk = i % DTK;
             const bool in = k0 + kk < d.k;
-            sw[kk][r] = in && n0 + r < d.n ? to_f32(((const W *)d.w)[(n0 + r) * d.k + k0 + kk]) : 0.0f;
+            sw[kk][r] = in && n0 + r < d.n ? to_f32(((const W *)d.w)[(n0 + r) * d.ldw + k0 + kk]) : 0.0f;
             sx[kk][r] = in && m0 + r < d.m ? to_f32(((const X *)d.x)[(m0 + r) * d.ldx + k0 + kk]) : 0.0f;
         }
         __syncthreads();
@@ -216,9 +230,17 @@ dense_tiled_kernel(DenseMm d) {
     for (int i = 0; i < 4; i++)
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-            const int64_t row = n0 + tn + j, col = m0 + tm + i;
+            int64_t row = n0 + tn + j;
+            const int64_t col = m0 + tm + i;
             if (row >= d.n || col >= d.m) continue;
-            float v = dense_act(d.act, acc[i][j]);
+            float v = acc[i][j] + (d.bias ? d.bias[row] : 0.0f);
+            if (d.act == ACT_CLAMPED_GATE) {
+                if (j & 1) continue;
+                v = clamped_gate(v, acc[i][j | 1] + (d.bias ? d.bias[row + 1] : 0.0f), d.act_limit, d.act_alpha);
+                row >>= 1;
+            } else {
+                v = dense_act(d.act, v);
+            }
             if (d.addend) v += d.addend[col * d.ld_addend + row];
             if (d.y_type == B200_TYPE_F32) ((float *)d.y)[col * d.ldy + row] = v;
             else ((__nv_bfloat16 *)d.y)[col * d.ldy + row] = __float2bfloat16_rn(v);
@@ -297,6 +319,8 @@ bool dense_type(int t) { return t == B200_TYPE_F32 || t == B200_TYPE_BF16; }
 int launch_dense_mm(const DenseMm &d, cudaStream_t s) {
     B200_REQUIRE(d.w && d.x && d.y && dense_type(d.w_type) && dense_type(d.x_type) && dense_type(d.y_type), "dense mat-mul: operands must be F32 or BF16");
     B200_REQUIRE(d.n > 0 && d.k > 0 && d.m >= 0 && d.k < (1ll << 31) && d.m < (1ll << 31), "dense mat-mul: bad shape");
+    B200_REQUIRE(d.ldw >= d.k, "dense mat-mul: weight rows overlap");
+    B200_REQUIRE(d.act != ACT_CLAMPED_GATE || (d.n % 2 == 0 && d.addend == nullptr), "dense mat-mul: a gated result takes pairs of rows and no addend");
     if (d.m == 0) return B200_STATUS_SUCCESS;
     if (d.m <= DENSE_FEW_ROWS && d.x_type == B200_TYPE_F32) return d.w_type == B200_TYPE_F32 ? launch_few<float>(d, s) : launch_few<__nv_bfloat16>(d, s);
     B200_REQUIRE(d.norm_w == nullptr, "dense mat-mul: the norm rides along with up to %d F32 rows only", DENSE_FEW_ROWS);

@@ -1,10 +1,11 @@
-// BF16 x BF16 mat-mul on the tensor cores for many activation rows: y[m][n] = act(w[n][k] x[m][k]) + addend, F32 sums.
+// BF16 x BF16 mat-mul on the tensor cores for many activation rows: y[m][n] = act(w[n][k] x[m][k] + bias) + addend, F32 sums.
 //
 // Output tiles of 128 weight rows x NC activation rows (64, 128 or 256), walked by persistent CTAs, one per SM, the column blocks of a
 // weight row block next to each other so that the weights cross HBM once.  Per tile a pipeline of K = 64 steps: one thread moves the
 // two operand boxes with TMA (128-byte swizzle; the hardware fills what lies outside either matrix with zeros), one thread issues four
 // M 128 x N NC x K 16 MMAs per step into one of two tensor-memory stages, four warps drain the other stage: lane = weight row, so a
-// store of one activation row's 32 outputs is one contiguous piece.  The activation function and the residual add are done there.
+// store of one activation row's 32 outputs is one contiguous piece.  The activation function and the residual add are done there;
+// a gated one takes neighbouring weight rows (gate, up), which neighbouring lanes exchange, each keeping every other activation row.
 // Every wait is bounded; a wait that runs out raises the CTA's abort flag and the device error word.
 #include <cuda.h>
 
@@ -37,7 +38,9 @@ struct GbOut {
     int64_t ldy;
     const float *addend;
     int64_t ld_addend;
+    const float *bias;
     int act;
+    float act_limit, act_alpha;
     int n, m;
 };
 
@@ -187,6 +190,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int row = rb * GB_ROWS + 32 * q + lane, col0 = cb * NC;
             const bool row_ok = row < o.n;
+            const float bias = o.bias && row_ok ? o.bias[row] : 0.0f;
             const uint32_t trow = tmem + ((uint32_t)(32 * q) << 16) + (uint32_t)(ts * NC);
 #pragma unroll 1
             for (int c0 = 0; c0 < NC; c0 += 32) {
@@ -206,12 +210,26 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_
                     __syncwarp();
                     if (lane == 0) gb_bar_arrive(gb_smem(&bars.tempty[ts]));
                 }
+                if (o.act == ACT_CLAMPED_GATE) {
+                    const int odd = lane & 1;
+#pragma unroll
+                    for (int c = 0; c < 32; c += 2) {
+                        const float x0 = __uint_as_float(v[c]) + bias, x1 = __uint_as_float(v[c + 1]) + bias;
+                        const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
+                        const float r = clamped_gate(odd ? other : x0, odd ? x1 : other, o.act_limit, o.act_alpha);
+                        const int col = col0 + c0 + c + odd;
+                        if (!row_ok || col >= o.m) continue;
+                        if (o.y_type == B200_TYPE_F32) ((float *)o.y)[(int64_t)col * o.ldy + (row >> 1)] = r;
+                        else ((__nv_bfloat16 *)o.y)[(int64_t)col * o.ldy + (row >> 1)] = __float2bfloat16_rn(r);
+                    }
+                    continue;
+                }
                 if (!row_ok) continue;
 #pragma unroll
                 for (int c = 0; c < 32; c++) {
                     const int col = col0 + c0 + c;
                     if (col >= o.m) break;
-                    float r = dense_act(o.act, __uint_as_float(v[c]));
+                    float r = dense_act(o.act, __uint_as_float(v[c]) + bias);
                     if (o.addend) r += ad[c];
                     if (o.y_type == B200_TYPE_F32) ((float *)o.y)[(int64_t)col * o.ldy + row] = r;
                     else ((__nv_bfloat16 *)o.y)[(int64_t)col * o.ldy + row] = __float2bfloat16_rn(r);
@@ -265,7 +283,7 @@ int launch_nc(const DenseMm &d, int sms, cudaStream_t s) {
         attr_done[dev] = true;
     }
     CUtensorMap wmap, xmap;
-    int rc = rows_map(&wmap, d.w, d.k, d.n, d.k, GB_ROWS);
+    int rc = rows_map(&wmap, d.w, d.k, d.n, d.ldw, GB_ROWS);
     if (rc == B200_STATUS_SUCCESS) rc = rows_map(&xmap, d.x, d.k, d.m, d.ldx, NC);
     if (rc != B200_STATUS_SUCCESS) return rc;
     int *err = nullptr;
@@ -273,7 +291,7 @@ int launch_nc(const DenseMm &d, int sms, cudaStream_t s) {
     if (rc != B200_STATUS_SUCCESS) return rc;
     const int64_t rb = (d.n + GB_ROWS - 1) / GB_ROWS, cb = (d.m + NC - 1) / NC;
     B200_REQUIRE(rb * cb < (1ll << 31), "gemm: too many tiles");
-    const GbOut o = {d.y, d.y_type, d.ldy, d.addend, d.ld_addend, d.act, (int)d.n, (int)d.m};
+    const GbOut o = {d.y, d.y_type, d.ldy, d.addend, d.ld_addend, d.bias, d.act, d.act_limit, d.act_alpha, (int)d.n, (int)d.m};
     const int tiles = (int)(rb * cb);
     return launch_pdl(gemm_bf16_tcgen05_kernel<NC>, dim3((unsigned)(tiles < sms ? tiles : sms)), dim3(GB_THREADS), (size_t)C::SMEM, s, wmap, xmap, o,
                       (int)((d.k + GB_K - 1) / GB_K), (int)cb, tiles, err);
@@ -283,7 +301,7 @@ int launch_nc(const DenseMm &d, int sms, cudaStream_t s) {
 
 // what the tensor maps can describe: 16-byte aligned bases and row strides
 bool gemm_bf16_takes(const DenseMm &d) {
-    return d.w_type == B200_TYPE_BF16 && d.x_type == B200_TYPE_BF16 && d.k % 8 == 0 && d.ldx % 8 == 0 && (((uintptr_t)d.w | (uintptr_t)d.x) & 15) == 0 &&
+    return d.w_type == B200_TYPE_BF16 && d.x_type == B200_TYPE_BF16 && d.k % 8 == 0 && d.ldx % 8 == 0 && d.ldw % 8 == 0 && (((uintptr_t)d.w | (uintptr_t)d.x) & 15) == 0 &&
            d.n < (1ll << 31) - 256 && d.m < (1ll << 31) - 256 && d.norm_w == nullptr;
 }
 

@@ -12,7 +12,7 @@
 //   latent_attn_mma_kernel  64 rows x 64-key tiles on mma.sync (BF16 operands, F32 scores and sums; a weight goes in as two BF16
 //                           parts, so that it keeps its 32-bit value to 2^-17), or
 //   latent_attn_kernel      a warp per (row, head), F32 arithmetic, any type and size
-#include "dense.cuh"
+#include "attn_tile.cuh"
 
 namespace b200 {
 
@@ -22,7 +22,6 @@ constexpr int LT = 256;             // threads per block
 constexpr int LK = 32, LH = 8;      // keys per tile, heads (one per warp) per block of the few-rows kernel
 constexpr int LRB = 512;            // latent elements a block of it accumulates
 constexpr int LV_ROWS = 32;         // value rows per block of the merge
-constexpr int ERR_CELL = 2, ERR_POS = 3;
 
 // element j of a rotated part at x, by the position's row of (cos, sin) pairs
 __device__ __forceinline__ float rotated(const float *x, const float *rope, int rot_dims, int j) {
@@ -136,16 +135,8 @@ latent_query_kernel(LatentArgs a, int lanes, int *err) {
         for (int j = tid; j < a.rot; j += LT) out[a.rank + j] = rotated(q + a.dim, rope, a.rot_dims, j);
 }
 
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
-
 // the keys a row sees: positions [lo, hi]
 __device__ __forceinline__ int first_key(const LatentArgs &a, int pos) { return a.window > 0 ? max(0, pos - a.window + 1) : 0; }
-
-// shared-memory row of a key in 16-byte units: odd, so that eight lanes reading eight rows touch different banks
-template <typename T>
-__host__ __device__ inline int key_units(int n) { return ((n * (int)sizeof(T) + 15) / 16) | 1; }
 
 template <typename T>
 __global__ void __launch_bounds__(LT)
@@ -329,23 +320,6 @@ latent_value_kernel(LatentArgs a) {
 }
 
 // ---- many rows ---------------------------------------------------------------------------------------------
-// tile ti of 64 (or `per`) rows -> its segment, first row inside it and rows; false past the last
-__device__ __forceinline__ const int32_t *find_tile(const LatentArgs &a, int per, int ti, int *r0, int *rows, int *err) {
-    for (int s = 0; s < (int)a.n_seg; s++) {
-        const int32_t *sg = a.seg + s * SEG_FIELDS;
-        const int n = sg[SEG_ROWS], k = (n + per - 1) / per;
-        if (ti < k) {
-            *r0 = ti * per;
-            *rows = min(per, n - ti * per);
-            if (sg[SEG_ROW0] >= 0 && (int64_t)sg[SEG_ROW0] + n <= a.n) return sg;
-            atomicExch(err, ERR_SEGMENT);
-            return nullptr;
-        }
-        ti -= k;
-    }
-    return nullptr;
-}
-
 template <typename T, typename Y>
 __global__ void __launch_bounds__(LT)
 latent_attn_kernel(LatentArgs a, int *err) {
@@ -355,7 +329,7 @@ latent_attn_kernel(LatentArgs a, int *err) {
     pdl_trigger();
     pdl_wait();
     int r0, rows;
-    const int32_t *sg = find_tile(a, LT / 32, blockIdx.x, &r0, &rows, err);
+    const int32_t *sg = find_tile(a.seg, a.n_seg, a.n, LT / 32, blockIdx.x, &r0, &rows, err);
     if (!sg || warp >= rows) return;
     const int64_t row = sg[SEG_ROW0] + r0 + warp;
     const int pos = sg[SEG_POS0] + r0 + warp, lo = first_key(a, pos);
@@ -404,18 +378,6 @@ latent_attn_kernel(LatentArgs a, int *err) {
 }
 
 // tensor-core form: 4 warps x 16 rows, DK = dim + rot and DV = vdim padded
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
-}
-
 constexpr int MT = 128, MQ = 64, MK = 64;
 
 // One buffer each for keys and values: the next keys land while the weights meet the values, the next values while the queries meet
@@ -432,7 +394,7 @@ latent_attn_mma_kernel(LatentArgs a, int *err) {
     pdl_wait();
     int r0, rows;
     // later tiles of a prompt see more keys: they go first
-    const int32_t *sg = find_tile(a, MQ, gridDim.x - 1 - blockIdx.x, &r0, &rows, err);
+    const int32_t *sg = find_tile(a.seg, a.n_seg, a.n, MQ, gridDim.x - 1 - blockIdx.x, &r0, &rows, err);
     if (!sg) return;
     const int64_t row0 = sg[SEG_ROW0] + r0;
     const int pos0 = sg[SEG_POS0] + r0, last = pos0 + rows - 1;

@@ -130,6 +130,7 @@ static int llama_new_impl(const b200_llama_hparams *hp, int device, int32_t n_ct
 // ---- architectures described by a configuration file -------------------------------------------------------
 static const struct { const char *name; ArchFromConfig from_config; } CONFIG_ARCHS[] = {
     {"Rukusun", rukusun_from_config},
+    {"Lenolix", lenolix_from_config},
 };
 
 int b200_model_new(const char *config_json, int dtype, int device, int32_t n_ctx, int32_t n_batch, int32_t n_seq, b200_llama **out) {
@@ -236,7 +237,15 @@ static int set_placed_tensor(b200_llama *c, const char *name, int type, int64_t 
         src = h.data();
     }
     c->backend->iface.synchronize(c->backend);
-    t->buffer->iface.set_tensor(t->buffer, t, src, offset, count * plain_type_size(p.type));
+    if (p.row_step == 1) {
+        t->buffer->iface.set_tensor(t->buffer, t, src, offset, count * plain_type_size(p.type));
+    } else {   // between rows of other tensors: what is there comes to the host and goes back
+        const size_t row = t->nb[1], span = row * (size_t)((p.rows - 1) * p.row_step + 1);
+        c->shard_tmp.resize(span);
+        t->buffer->iface.get_tensor(t->buffer, t, c->shard_tmp.data(), offset, span);
+        for (int64_t r = 0; r < p.rows; r++) memcpy(&c->shard_tmp[row * (size_t)(r * p.row_step)], (const uint8_t *)src + row * (size_t)r, row);
+        t->buffer->iface.set_tensor(t->buffer, t, c->shard_tmp.data(), offset, span);
+    }
     c->tensors_set.insert(name);
     c->graphs.clear();
     c->last = nullptr;
@@ -334,7 +343,7 @@ int b200_llama_decode(b200_llama *c, const int32_t *tokens, const int32_t *pos, 
 
 // A step of a segmented architecture, on the host: the sequences among its rows, checked (a sequence's rows stand together and
 // continue it), then their cells and slots, and the inputs the nodes read.  Nothing changes before every check has passed.
-static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_ids, int32_t n, StepShape *s) {
+static int plan_segments(b200_llama *c, const int32_t *tokens, const int32_t *pos, const int32_t *seq_ids, int32_t n, StepShape *s) {
     struct Seg { int32_t seq, row0, rows; int64_t pos0; };
     std::vector<Seg> segs;
     for (int32_t i = 0; i < n; i++) {
@@ -351,7 +360,7 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
         B200_REQUIRE(pos[i] == want, "llama_decode: sequence %d continues at position %lld, not %d", q, (long long)want, pos[i]);
         segs.push_back({q, i, 1, pos[i]});
     }
-    const int64_t span = c->arch->key_span();
+    const int64_t span = c->arch->key_span(), keep = span > 0 ? c->arch->kept_first() : 0;
     int64_t fresh = 0, free_slots = 0;
     for (const Seg &g : segs) fresh += c->seqs.find(g.seq) == c->seqs.end();
     for (int32_t q : c->slot_seq) free_slots += q < 0;
@@ -361,6 +370,7 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
     c->seg_host.assign(segs.size() * SEG_FIELDS, 0);
     c->row_seg_host.assign(n, 0);
     c->cells_host.assign(n, 0);
+    c->prev_host.assign(n, -1);
     c->tab_host.clear();
     int64_t max_keys = 1, max_rows = 1;
     for (size_t k = 0; k < segs.size(); k++) {
@@ -370,6 +380,7 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
         if (is_new) {
             q.slot = (int32_t)(std::find(c->slot_seq.begin(), c->slot_seq.end(), -1) - c->slot_seq.begin());
             c->slot_seq[q.slot] = g.seq;
+            q.kept = keep;
         }
         int32_t *f = &c->seg_host[k * SEG_FIELDS];
         f[SEG_ROW0] = g.row0;
@@ -379,6 +390,8 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
         f[SEG_POS0] = (int32_t)g.pos0;
         for (int32_t i = 0; i < g.rows; i++) {
             c->row_seg_host[g.row0 + i] = (int32_t)k;
+            c->prev_host[g.row0 + i] = q.last_token;
+            q.last_token = tokens[g.row0 + i];
             if (span < 0) continue;
             int32_t cell = c->first_free;
             while (c->cell_seq[cell] >= 0) cell++;
@@ -388,17 +401,19 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
             c->used++;
             c->high = std::max(c->high, cell + 1);
             c->cells_host[g.row0 + i] = cell;
-            q.cells.push_back(cell);
+            (g.pos0 + i < keep ? q.first_cells : q.cells).push_back(cell);
         }
         q.next_pos = g.pos0 + g.rows;
         max_rows = std::max<int64_t>(max_rows, g.rows);
         if (span >= 0) {
-            // the positions the first row can see, up to the last row's own
-            const int64_t key0 = span > 0 ? std::max<int64_t>(0, g.pos0 - span + 1) : 0;
-            f[SEG_TAB0] = (int32_t)c->tab_host.size();
+            // the positions the first row can see, up to the last row's own, behind the ones that are kept for good
+            const int64_t key0 = span > 0 ? std::max<int64_t>(keep, g.pos0 - span + 1) : 0, at = (int64_t)c->tab_host.size();
+            f[SEG_TAB0] = (int32_t)at;
             f[SEG_KEY0] = (int32_t)key0;
+            f[SEG_KEPT] = (int32_t)q.first_cells.size();
+            c->tab_host.insert(c->tab_host.end(), q.first_cells.begin(), q.first_cells.end());
             for (int64_t p = key0; p < q.next_pos; p++) c->tab_host.push_back(q.cells[p - q.kept]);
-            max_keys = std::max(max_keys, q.next_pos - key0);
+            max_keys = std::max(max_keys, (int64_t)c->tab_host.size() - at);
         }
     }
     s->n_seg = (int64_t)segs.size();
@@ -406,7 +421,7 @@ static int plan_segments(b200_llama *c, const int32_t *pos, const int32_t *seq_i
     while (s->max_rows < max_rows) s->max_rows *= 2;
     if (span >= 0) {
         s->n_tab = std::min<int64_t>(((int64_t)c->tab_host.size() + KV_PAD - 1) / KV_PAD * KV_PAD, (c->n_ctx + KV_PAD - 1) / KV_PAD * KV_PAD);
-        if (max_rows == 1 && span > 0) max_keys = std::min(max_keys, span);
+        if (max_rows == 1 && span > 0) max_keys = std::min(max_keys, span + keep);
         s->max_keys = std::min<int64_t>((max_keys + KV_PAD - 1) / KV_PAD * KV_PAD, s->n_tab);
         c->tab_host.resize(s->n_tab, 0);
     }
@@ -451,7 +466,7 @@ int b200_llama_decode_seqs(b200_llama *c, const int32_t *tokens, const int32_t *
         }
         shape.n_kv = n_kv_for(c, high);
     } else {
-        int rc = plan_segments(c, pos, seq_ids, n, &shape);
+        int rc = plan_segments(c, tokens, pos, seq_ids, n, &shape);
         if (rc != B200_STATUS_SUCCESS) return rc;
     }
 
@@ -502,6 +517,7 @@ int b200_llama_decode_seqs(b200_llama *c, const int32_t *tokens, const int32_t *
     c->backend->iface.synchronize(c->backend);
     set_input_async(c->backend, g->tokens, tokens, (size_t)n * 4);
     set_input_async(c->backend, g->pos, pos, (size_t)n * 4);
+    if (g->prev) set_input_async(c->backend, g->prev, c->prev_host.data(), (size_t)n * 4);
     if (masked) {
         set_input_async(c->backend, g->mask, c->mask_host.data(), c->mask_host.size() * 2);
         set_input_async(c->backend, g->row_idx, c->idx_host.data(), (size_t)n * 8);
