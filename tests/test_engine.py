@@ -100,3 +100,31 @@ def test_configurations_that_describe_no_model_are_refused():
     assert "tau" in refused(lambda c: c["layers"][0]["mixer"].update(tau=0))
     assert "dense" in refused(lambda c: c["layers"][1]["mlp"].update(kind="other"))
     assert "rotated" in refused(lambda c: c["layers"][1]["mixer"]["rot"].update(dims=7))
+
+
+def test_lenolix_configurations_that_describe_no_model_are_refused():
+    import lenolix_models as M
+    mod = b200.load()
+    ll = importlib.import_module("llama_rust_b200.llama")
+
+    def refused(change):
+        cfg = M.config([M.layer(), M.layer()], loop=(0, 1, 2))
+        change(cfg)
+        with pytest.raises(mod.B200Error) as e:
+            ll.Model(cfg, 256, 32)
+        return str(e.value)
+
+    mixer = lambda c: c["layers"][1]["mixer"]  # noqa: E731
+    assert "kv_heads" in refused(lambda c: mixer(c).pop("kv_heads"))
+    assert "multiple of kv_heads" in refused(lambda c: mixer(c).update(kv_heads=3))
+    assert "not known" in refused(lambda c: c["layers"][0].update(type="gla"))
+    assert "rotated" in refused(lambda c: mixer(c)["rot"].update(dims=7))
+    assert "rotated" in refused(lambda c: mixer(c)["rot"].update(dims=22))
+    assert "scaling" in refused(lambda c: mixer(c)["rot"]["scaling"].update(factor=0))
+    assert "mask" in refused(lambda c: mixer(c)["mask"].update(size=0))
+    assert "keep_first" in refused(lambda c: mixer(c)["mask"].update(keep_first=-1))
+    assert "limit" in refused(lambda c: c["layers"][0]["mlp"].pop("limit"))
+    assert "dense" in refused(lambda c: c["layers"][0]["mlp"].update(kind="other"))
+    assert "buckets" in refused(lambda c: c["embedding"]["bigram"].update(buckets=0))
+    assert "bigram" in refused(lambda c: c["embedding"]["bigram"].update(mul_cur=1.5))
+    assert "loop" in refused(lambda c: c["loop"].update(stop=3))

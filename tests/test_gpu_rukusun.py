@@ -4,7 +4,6 @@ serving loop, model folders."""
 import importlib
 import json
 import os
-import struct
 import subprocess
 import sys
 
@@ -14,28 +13,9 @@ import pytest
 import b200
 import plain_decoder as P
 import rukusun_models as M
+from decoder_checks import Expected, check, cycle, feed, model, plain_greedy, write_folder
 
 pytestmark = pytest.mark.gpu
-
-TOL = 2e-5   # F32 models: of the logits' spread (M.error)
-
-
-class Expected:
-    """the plain decoder's logits of a sequence, and per row how far BF16 rounding alone moves them (two ways of rounding: some
-    rows of random models are far more sensitive than others)"""
-
-    def __init__(self, cfg, w, toks, dtype="float32"):
-        self.rows = P.Plain(cfg, w).feed(toks)
-        self.limit = np.full(len(toks), TOL)
-        if dtype == "bfloat16":
-            shaken = [M.error(P.Plain(cfg, w, lambda x, f=f: M.bf16(x * f) / f).feed(toks), self.rows) for f in (1.0, 1.37)]
-            self.limit = 1e-2 + 3.0 * np.maximum(*shaken)
-
-    def __getitem__(self, at):
-        part = object.__new__(Expected)
-        part.rows, part.limit = self.rows[at], self.limit[at]
-        return part
-
 
 @pytest.fixture(scope="module")
 def ll():
@@ -46,34 +26,6 @@ def ll():
 @pytest.fixture(scope="module")
 def engine(ll):
     return importlib.import_module("llama_rust_b200.engine")
-
-
-def model(ll, cfg, w, dtype="float32", n_ctx=512, n_batch=512, n_seq=4):
-    m = ll.Model(cfg, n_ctx, n_batch, n_seq=n_seq, dtype=dtype)
-    m.set_tensors(w)
-    return m
-
-
-def feed(m, toks, sizes, seq=0, at=0):
-    """the tokens in portions; logits of every one"""
-    out, i = [], 0
-    while i < len(toks):
-        n = min(next(sizes) if not isinstance(sizes, int) else sizes, len(toks) - i)
-        got, _ = m.decode_seqs(toks[i:i + n], np.arange(at + i, at + i + n), [seq] * n, np.arange(n))
-        out.append(got)
-        i += n
-    return np.concatenate(out)
-
-
-def cycle(*sizes):
-    while True:
-        yield from sizes
-
-
-def check(got, want, what=""):
-    e = M.error(got, want.rows)
-    worst = int((e / want.limit).argmax())
-    assert (e < want.limit).all(), f"{what}: row {worst} is {e[worst]:.2e} away ({want.limit[worst]:.2e} allowed)"
 
 
 STACK = [M.gla(), M.latent(), M.gla(heads=1, dim=32, vdim=8, tau=1.0, ff=0)]
@@ -317,18 +269,6 @@ def test_long_decoding(ll):
     check(feed(m, toks, cycle(60, *[1] * 360)), want)
 
 
-def plain_greedy(cfg, w, prompt, n):
-    p, out = P.Plain(cfg, w), []
-    row = p.feed(prompt)[-1]
-    gap = np.inf
-    for _ in range(n):
-        s = np.sort(row)
-        gap = min(gap, (s[-1] - s[-2]) / row.std())
-        out.append(int(row.argmax()))
-        row = p.feed([out[-1]])[-1]
-    return out, gap
-
-
 @pytest.mark.parametrize("portion,max_seqs", [(None, 8), (5, 2)])
 def test_generation_through_the_serving_loop(ll, engine, portion, max_seqs):
     cfg = M.config(STACK, loop=(1, 3, 2))
@@ -340,20 +280,6 @@ def test_generation_through_the_serving_loop(ll, engine, portion, max_seqs):
         want, gap = plain_greedy(cfg, w, p, 12)
         assert gap > 1e-4 and g == want
     assert m.kv_used() == 0
-
-
-def write_folder(path, cfg, w):
-    table, at, parts = {"__metadata__": {"format": "pt"}}, 0, []
-    for k, v in w.items():
-        raw = (np.ascontiguousarray(v, np.float32).view(np.uint32) >> 16).astype(np.uint16).tobytes()
-        table[k] = {"dtype": "BF16", "shape": list(v.shape), "data_offsets": [at, at + len(raw)]}
-        at += len(raw)
-        parts.append(raw)
-    head = json.dumps(table).encode()
-    with open(os.path.join(path, "model.safetensors"), "wb") as f:
-        f.write(struct.pack("<Q", len(head)) + head + b"".join(parts))
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f)
 
 
 def test_programs_over_a_model_folder(tmp_path, ll):
