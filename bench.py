@@ -1030,7 +1030,7 @@ def case_llama(args):
 
 # Layers the size of a real model's, by width: the design's two kinds in the proportion 3 : 1, and the llama model of the
 # same width and the same number of weights per layer (its FFN size makes up the difference)
-RUKUSUN_VOCAB = 32000
+DESIGN_VOCAB = 32000
 
 
 def rukusun_config(width, layers, window=1024):
@@ -1039,21 +1039,63 @@ def rukusun_config(width, layers, window=1024):
            "mixer": {"heads": width // 128, "dim": 128, "rot_dim": 64, "kv_rank": 512, "vdim": 128, "mask": {"size": window}, "scale": 192 ** -0.5,
                      "rot": {"base": 10000.0, "dims": 64}}}
     return {"architecture": "Rukusun", "embedding": {"scale": float(width) ** 0.5}, "layers": [lat if i % 4 == 3 else gla for i in range(layers)],
-            "norm": {"eps": 1e-5}, "vocab": RUKUSUN_VOCAB, "width": width}
+            "norm": {"eps": 1e-5}, "vocab": DESIGN_VOCAB, "width": width}
 
 
-def rukusun_tensors(cfg, rank=16):
-    """(name, BF16 bits) of every tensor: seeded normals of the right spread, large matrices repeat a block of rows"""
-    rng = np.random.default_rng(0)
-    base = rng.standard_normal(1 << 20).astype(np.float32)
-    E, V = cfg["width"], cfg["vocab"]
+def lenolix_config(width, layers, window=1024, keep=64, loop=None):
+    """weights per layer as many as Rukusun's of the same width: the feed-forward makes up the difference"""
+    heads, groups = width // 128, max(1, width // 512)
+    attn = (2 * heads + 2 * groups) * 128
+    ff = round((12 * width - attn) / 3 / 128) * 128
+    lay = {"type": "attention", "mlp": {"kind": "dense", "ff": ff, "limit": 7.0},
+           "mixer": {"heads": heads, "kv_heads": groups, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window, "keep_first": keep},
+                     "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    return {"architecture": "Lenolix", "embedding": {"scale": float(width) ** 0.5, "bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 17}}, "layers": [lay] * layers,
+            "loop": loop, "norm": {"eps": 1e-5}, "vocab": DESIGN_VOCAB, "width": width}
+
+
+def bf16_tensors():
+    """mat(n, k, gain, mean), vec(n, mean, dev) -> BF16 bits: seeded normals of the right spread, large matrices repeat a block of rows"""
+    base = np.random.default_rng(0).standard_normal(1 << 20).astype(np.float32)
 
     def mat(n, k, gain=1.0, mean=0.0):
         block = (base * (gain / np.sqrt(k)) + mean).astype(np.float32).view(np.uint32)
         return np.resize(((block + 0x8000) >> 16).astype(np.uint16), (n, k))
 
-    def vec(n, mean, dev):
-        return mat(1, n, dev * np.sqrt(n), mean).reshape(n)
+    return mat, lambda n, mean, dev: mat(1, n, dev * np.sqrt(n), mean).reshape(n)
+
+
+def lenolix_tensors(cfg):
+    """(name, BF16 bits) of every tensor"""
+    mat, vec = bf16_tensors()
+    E = cfg["width"]
+    yield "embed", mat(cfg["vocab"], E)
+    yield "bigram", mat(cfg["embedding"]["bigram"]["buckets"] + 1, E)
+    if cfg["loop"]:
+        yield "loop.in", mat(E, 2 * E)
+        yield "loop.step", mat(cfg["loop"]["times"], E, 0.1)
+    for i, lay in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", lay["mixer"], lay["mlp"]["ff"]
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            yield p + n, vec(E, 1.0, 0.1)
+            yield p + n + ".b", vec(E, 0.0, 0.1)
+        for n in ("ls1", "ls2"):
+            yield p + n, vec(E, 0.5, 0.1)
+        for n, rows in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+            yield p + "mix." + n, mat(rows, E)
+        yield p + "mix.sink", vec(m["heads"], 0.0, 1.0)
+        yield p + "mix.o", mat(E, m["heads"] * m["vdim"])
+        yield p + "mlp.gate", mat(ff, E)
+        yield p + "mlp.up", mat(ff, E)
+        yield p + "mlp.down", mat(E, ff)
+    yield "final.norm", vec(E, 1.0, 0.1)
+    yield "final.norm.b", vec(E, 0.0, 0.1)
+
+
+def rukusun_tensors(cfg, rank=16):
+    """(name, BF16 bits) of every tensor"""
+    mat, vec = bf16_tensors()
+    E, V = cfg["width"], cfg["vocab"]
 
     yield "embed", mat(V, E)
     yield "head", mat(V, E)
@@ -1084,15 +1126,21 @@ def rukusun_tensors(cfg, rank=16):
             yield p + "mix.g", mat(H, E)
 
 
-def build_rukusun(width, layers, n_ctx, n_batch, n_seq=16):
+DESIGNS = {"rukusun": (rukusun_config, rukusun_tensors), "lenolix": (lenolix_config, lenolix_tensors)}
+
+
+def build_design(design, width, layers, n_ctx, n_batch, n_seq=16, **cfg_args):
+    """-> the model, its configuration, the weights a step's mat-muls read"""
     load_pkg()
     ll = importlib.import_module("llama_rust_b200.llama")
-    cfg = rukusun_config(width, layers)
+    make, tensors = DESIGNS[design]
+    cfg = make(width, layers, **cfg_args)
     gpu = ll.Model(cfg, n_ctx, n_batch, n_seq=n_seq)
+    tied = not any(name == "head" for name, _ in tensors(dict(cfg, layers=[])))
     weights = 0
-    for name, t in rukusun_tensors(cfg):
+    for name, t in tensors(cfg):
         gpu.set_tensors({name: t})
-        if ".mix.norm" not in name and name != "embed":
+        if t.ndim == 2 and name != "bigram" and (name != "embed" or tied):
             weights += t.size
     return gpu, cfg, weights
 
@@ -1104,7 +1152,7 @@ def build_equal_llama(width, layers, weights_per_layer, n_ctx, n_batch):
     syn = load_standalone("synth")
     attn = 2 * width * width + 2 * width * 1024
     ff = max(256, round((weights_per_layer - attn) / (3 * width) / 256) * 256)
-    hp = dict(sh.LLAMA3_8B, n_vocab=RUKUSUN_VOCAB, n_embd=width, n_head=width // 128, n_head_kv=8, n_ff=ff, n_layer=layers)
+    hp = dict(sh.LLAMA3_8B, n_vocab=DESIGN_VOCAB, n_embd=width, n_head=width // 128, n_head_kv=8, n_ff=ff, n_layer=layers)
     gpu = ll.Llama(hp, n_ctx, n_batch)
     for name, ty, arr, ne0, ne1 in syn.llama_tensors(hp, lambda n: sh.q4_k_m_type(n, layers), tensor_shapes=sh.tensor_shapes):
         gpu.set_tensor(name, ty, arr, ne0, ne1)
@@ -1132,20 +1180,24 @@ def time_model(gpu, vocab, prompt, steps):
     return out
 
 
-def case_rukusun(args):
-    """`--case rukusun`: prefill and decode throughput of the design at a few widths, beside a llama model of equal size (Q4_K_M,
-    fast numerics).  `rukusun_pp` / `rukusun_tg`: one prompt / R single-token steps of a small model, eager launches."""
-    small = args.case != "rukusun"
+def case_design(args):
+    """`--case rukusun` / `lenolix`: prefill and decode throughput of the design at a few widths, beside models of equal size: llama
+    (Q4_K_M, fast numerics) and, for Lenolix, Rukusun.  `.._pp` / `.._tg`: one prompt / R single-token steps of a small model, eager
+    launches."""
+    design = args.case.split("_")[0]
+    small = args.case != design
     if small:
         os.environ["B200_CUDA_GRAPHS"] = "0"
     b = load_pkg()
     b.set_device(0)
     prompt = args.prompt if args.prompt > 16 else 2048
     if small:
-        gpu, cfg, _ = build_rukusun(args.width, args.layers if args.layers < 32 else 4, 2 * prompt, prompt)
+        layers = args.layers if args.layers < 32 else 4
+        more = {"loop": {"start": 0, "stop": 1, "times": 1}} if design == "lenolix" else {}
+        gpu, cfg, _ = build_design(design, args.width, layers, 2 * prompt, prompt, **more)
         toks = np.random.default_rng(0).integers(0, cfg["vocab"], prompt).astype(np.int32)
         tok = gpu.decode(toks, np.arange(prompt), logits=False, argmax=True)
-        if args.case == "rukusun_tg":
+        if args.case.endswith("_tg"):
             for i in range(args.launches):
                 tok = gpu.decode([tok], [prompt + i], logits=False, argmax=True)
         print(json.dumps({"case": args.case, "width": args.width, "kernel_error": b.kernel_error()}), flush=True)
@@ -1153,35 +1205,42 @@ def case_rukusun(args):
         return
     layers, steps = args.layers if args.layers < 32 else 8, 64
     hbm, tensor = peak_hbm()[0], peak_tensor()[0]
+
+    def figures(times, body, step_bytes):
+        pp, pp_dev, tg, tg_dev = times
+        return {"prefill_tok_s": prompt / pp_dev * 1e3, "prefill_e2e_tok_s": prompt / pp * 1e3, "decode_tok_s": 1e3 / tg_dev, "decode_e2e_tok_s": 1e3 / tg,
+                "prefill_of_tensor_peak": 2.0 * body * prompt / pp_dev / 1e9 / tensor, "decode_of_hbm_peak": step_bytes / tg_dev / 1e6 / hbm}
+
     rows = []
     for width in (1024, 2048, 4096):
-        mon = ClockSampler(0)
-        gpu, cfg, weights = build_rukusun(width, layers, 4096, prompt)
-        mon.start()
-        pp, pp_dev, tg, tg_dev = time_model(gpu, cfg["vocab"], prompt, steps)
-        clocks = mon.stop()
-        gpu.close()
-        head = cfg["vocab"] * width
-        lgpu, hp, lbytes = build_equal_llama(width, layers, (weights - head) / layers, 4096, prompt)
-        lpp, lpp_dev, ltg, ltg_dev = time_model(lgpu, hp["n_vocab"], prompt, steps)
+        row = {"width": width, "layers": layers, "prompt": prompt}
+        head = DESIGN_VOCAB * width
+        for name in [design] + (["rukusun"] if design != "rukusun" else []):
+            mon = ClockSampler(0)
+            gpu, cfg, weights = build_design(name, width, layers, 4096, prompt)
+            mon.start()
+            times = time_model(gpu, cfg["vocab"], prompt, steps)
+            row.setdefault("clocks", {})[name] = mon.stop()
+            gpu.close()
+            row[name] = dict(figures(times, weights - head, 2.0 * weights), weights_m=round(weights / 1e6))
+            if name == design:
+                own = weights
+        lgpu, hp, lbytes = build_equal_llama(width, layers, (own - head) / layers, 4096, prompt)
+        times = time_model(lgpu, hp["n_vocab"], prompt, steps)
         lgpu.close()
         lweights = hp["n_layer"] * (2 * width * width + 2 * width * 1024 + 3 * width * hp["n_ff"])
-        rows.append({
-            "width": width, "layers": layers, "prompt": prompt, "weights_m": round(weights / 1e6), "clocks": clocks,
-            "rukusun": {"prefill_tok_s": prompt / pp_dev * 1e3, "prefill_e2e_tok_s": prompt / pp * 1e3, "decode_tok_s": 1e3 / tg_dev, "decode_e2e_tok_s": 1e3 / tg,
-                        "prefill_of_tensor_peak": 2.0 * (weights - head) * prompt / pp_dev / 1e9 / tensor, "decode_of_hbm_peak": 2.0 * weights / tg_dev / 1e6 / hbm},
-            "llama_q4_k_m": {"n_ff": hp["n_ff"], "weights_m": round((lweights + head) / 1e6), "prefill_tok_s": prompt / lpp_dev * 1e3, "prefill_e2e_tok_s": prompt / lpp * 1e3,
-                             "decode_tok_s": 1e3 / ltg_dev, "decode_e2e_tok_s": 1e3 / ltg,
-                             "prefill_of_tensor_peak": 2.0 * lweights * prompt / lpp_dev / 1e9 / tensor, "decode_of_hbm_peak": lbytes / ltg_dev / 1e6 / hbm}})
-        note(json.dumps(rows[-1]))
-    print(json.dumps({"case": "rukusun", "data": "synthetic", "dtype": "bf16 weights, F32 residual", "sizes": rows, "kernel_error": b.kernel_error()}), flush=True)
+        row["llama_q4_k_m"] = dict(figures(times, lweights, lbytes), n_ff=hp["n_ff"], weights_m=round((lweights + head) / 1e6))
+        rows.append(row)
+        note(json.dumps(row))
+    print(json.dumps({"case": design, "data": "synthetic", "dtype": "bf16 weights, F32 residual", "sizes": rows, "kernel_error": b.kernel_error()}), flush=True)
 
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "fa", "llama_tg", "llama_pp", "llama_b16", "rukusun", "rukusun_pp", "rukusun_tg"],
-                    help="one small case for a profiler; rukusun: that design's throughput beside a llama model of equal size")
-    ap.add_argument("--width", type=int, default=4096, help="--case rukusun_pp / rukusun_tg: model width")
+    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "fa", "llama_tg", "llama_pp", "llama_b16", "rukusun", "rukusun_pp", "rukusun_tg", "lenolix", "lenolix_pp",
+                                                       "lenolix_tg"],
+                    help="one small case for a profiler; rukusun, lenolix: that design's throughput beside models of equal size")
+    ap.add_argument("--width", type=int, default=4096, help="--case .._pp / .._tg of a design: model width")
     ap.add_argument("--only", default="4096x4096", help="--case gemv / gemm: the shape NxK")
     ap.add_argument("--cols", type=int, default=512, help="--case gemm: activation rows")
     ap.add_argument("--wtype", default="Q4_K", choices=["Q4_K", "Q6_K"], help="--case gemm: weight type")
@@ -1207,8 +1266,8 @@ def main():
         return case_fa(args)
     if args.case == "gemm":
         return case_gemm(args)
-    if args.case and args.case.startswith("rukusun"):
-        return case_rukusun(args)
+    if args.case and args.case.split("_")[0] in DESIGNS:
+        return case_design(args)
     if args.case:
         return case_llama(args)
     rank, world, barrier, reduce_max = dist_setup(args.gpus)

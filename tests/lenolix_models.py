@@ -9,7 +9,7 @@ RAMP = {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 64}   # with base 50
 def layer(heads=4, kv_heads=2, dim=20, vdim=12, window=9, keep=3, scale=None, rot=8, base=500.0, scaling=RAMP, ff=40, limit=1.5):
     return {"type": "attention",
             "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale,
-                      "mask": {"size": window, "keep_first": keep} if window else None, "rot": {"base": base, "dims": rot, "scaling": scaling}},
+                      "mask": {"size": window, "keep_first": keep} if window else None, "rot": {"base": base, "dims": rot, "scaling": scaling and dict(scaling)}},
             "mlp": {"kind": "dense", "ff": ff, "limit": limit} if ff else None}
 
 
