@@ -22,9 +22,10 @@ namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr int GT = 256;            // threads per block
-constexpr int GK = 32;             // entries per tile of the few-rows kernel
+constexpr int GT = 256;            // threads per block, at most
+constexpr int GK = 16;             // entries per tile of a warp of the few-rows kernel
 constexpr int GH = 8;              // query heads per block of it
+constexpr int SPLITS_MAX = 8;      // blocks that share a row's entries
 
 __host__ __device__ inline int pad8(int n) { return (n + 7) / 8 * 8; }
 
@@ -109,38 +110,44 @@ struct Piece<float> {
     static __device__ __forceinline__ float2 pair(const float *p) { return *reinterpret_cast<const float2 *>(p); }
 };
 
-// shared memory of a block, in floats from the end of the tiles on
+// shared memory of a block of nw warps: each warp's own tiles (when they are done, the warps' sums), then floats at the offsets
 struct DecodeSmem {
-    int units, tile;                            // 16-byte units of an entry's row, bytes of a tile
-    int q, p, corr, red, out, ml, w, floats;    // offsets
-    __host__ __device__ DecodeSmem(int dim, int vdim, int es, int hw) {
+    int units, tile;                       // 16-byte units of an entry's row, bytes of a tile
+    size_t tiles;                          // bytes of the part ahead of the floats
+    int q, p, m, l, w, out, ml, floats;    // offsets
+    __host__ __device__ DecodeSmem(int dim, int vdim, int es, int hw, int nw, int stages) {
         const int d = pad8(dim), e = pad8(vdim);
-        units = ((d + e) * es / 16) | 1;
+        units = (d + e) * es / 16;
+        while (units % 4 != 2) units++;    // the two lanes of four neighbouring entries meet eight different bank groups
         tile = GK * units * 16;
-        int lanes = 1;
-        while (lanes < e / 2) lanes *= 2;
+        const size_t sums = (size_t)nw * hw * e * 4;
+        tiles = (size_t)nw * stages * tile;
+        if (tiles < sums) tiles = sums;
         q = 0;
         p = q + hw * d;
-        corr = p + GK * hw;
-        red = (corr + hw + 3) / 4 * 4;
-        out = red + (GT / (lanes < GT ? lanes : GT)) * hw * e;
+        m = p + nw * GK * hw;
+        l = m + nw * hw;
+        w = l + nw * hw;
+        out = (w + 8 * hw + 3) / 4 * 4;
         ml = out + hw * e;
-        w = ml + 2 * hw;
-        floats = w + 8 * hw;
+        floats = ml + 2 * hw;
     }
+    __host__ __device__ size_t bytes() const { return tiles + (size_t)floats * 4; }
 };
 
-template <typename T, int HW>
-__global__ void __launch_bounds__(GT)
+// A warp owns a stretch of the entries from load to weighted sum (no barrier until the end): two lanes share an entry's scores, then a
+// lane owns NP pairs of value channels.
+template <typename T, int HW, int NP>
+__global__ void __launch_bounds__(GT, 1)
 grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
-    constexpr int PE = Piece<T>::E, P = GH / HW;   // threads that share a (entry, head) dot product
+    constexpr int PE = Piece<T>::E;
     extern __shared__ __align__(16) uint8_t g_raw[];
     cg::cluster_group cluster = cg::this_cluster();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
     const int dim = pad8(a.dim), vdim = pad8(a.vdim), kp = dim / PE, vp = vdim / PE;
-    const DecodeSmem L(a.dim, a.vdim, (int)sizeof(T), HW);
-    float *f32 = (float *)(g_raw + (size_t)stages * L.tile);
-    float *sq = f32 + L.q, *sp = f32 + L.p, *scorr = f32 + L.corr, *sred = f32 + L.red, *sout = f32 + L.out, *sml = f32 + L.ml, *sw = f32 + L.w;
+    const DecodeSmem L(a.dim, a.vdim, (int)sizeof(T), HW, nw, stages);
+    float *f32 = (float *)(g_raw + L.tiles);
+    float *sq = f32 + L.q, *sp = f32 + L.p + warp * GK * HW, *sm = f32 + L.m, *sl = f32 + L.l, *sw = f32 + L.w, *sout = f32 + L.out, *sml = f32 + L.ml;
     const int rep = a.heads / a.kv_heads, g = blockIdx.y / head_groups, hg = blockIdx.y % head_groups, h0 = hg * GH, nh = min(HW, rep - h0);
     const int64_t row = blockIdx.z;
     pdl_trigger();
@@ -152,42 +159,50 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
         return;
     }
     const int32_t *sg = a.seg + (int64_t)si * SEG_FIELDS;
-    const int step0 = sg[SEG_POS0], step_n = sg[SEG_ROWS];
+    const int step0 = sg[SEG_POS0], step_n = sg[SEG_ROWS], step_row = sg[SEG_ROW0];
     const Entries en(a, pos, pos);
-    const int per = (en.total + GK * (int)gridDim.x - 1) / (GK * (int)gridDim.x) * GK, e0 = min(en.total, (int)blockIdx.x * per), e1 = min(en.total, e0 + per);
-    const int tiles = (e1 - e0 + GK - 1) / GK, head_row = dim + vdim;
+    const int owners = (int)gridDim.x * nw, per = (en.total + owners - 1) / owners;
+    const int e0 = min(en.total, ((int)blockIdx.x * nw + warp) * per), e1 = min(en.total, e0 + per), tiles = (e1 - e0 + GK - 1) / GK;
+    const int head_row = dim + vdim;
     const float *kx = a.proj + (int64_t)a.heads * a.dim + (int64_t)g * a.dim, *vx = a.proj + (int64_t)(a.heads + a.kv_heads) * a.dim + (int64_t)g * a.vdim;
-    // an entry's row: key channels, then value channels; a warp takes every eighth entry.  cells: those of earlier steps, fresh: this step's
-    const auto load_tile = [&](int t, bool cells, bool fresh) {
-        T *dst0 = (T *)(g_raw + (size_t)(t % stages) * L.tile);
-        for (int k = warp; k < GK; k += GT / 32) {
-            const int e = e0 + t * GK + k;
+    uint8_t *mine = g_raw + (size_t)warp * stages * L.tile;
+    // what stands behind entry lane % GK of tile t: a cell, -1 - r for row r of this step, NOTHING past the last or when the lists lack it
+    constexpr int64_t NOTHING = INT64_MIN;
+    const auto look_up = [&](int t) -> int64_t {
+        const int e = e0 + t * GK + lane % GK;
+        if (e >= e1) return NOTHING;
+        const int p = en.position(e);
+        if (p >= step0) {
+            if (p - step0 < step_n) return -1 - (int64_t)(step_row + (p - step0));
+            atomicExch(err, ERR_SEGMENT);
+            return NOTHING;
+        }
+        const int64_t cell = cell_of(a, sg, p);
+        if (cell < 0) atomicExch(err, ERR_CELL);
+        return cell < 0 ? NOTHING : cell;
+    };
+    // an entry's row: key channels, then value channels.  cells: those of earlier steps (what is missing is zero), fresh: this step's
+    const auto load_tile = [&](int t, int64_t found, bool cells, bool fresh) {
+        T *dst0 = (T *)(mine + (size_t)(t % stages) * L.tile);
+#pragma unroll 4
+        for (int k = 0; k < GK; k++) {
+            const int64_t at = __shfl_sync(0xffffffffu, found, k);
             T *dst = dst0 + (size_t)k * L.units * PE;
-            if (e >= e1) {
-                if (cells)
-                    for (int p = lane; p < kp + vp; p += 32) cp16(dst + p * PE, a.cache, false);
-                continue;
-            }
-            const int p = en.position(e);
-            if (p < step0) {
+            if (at >= 0 || at == NOTHING) {
                 if (!cells) continue;
-                const int64_t cell = cell_of(a, sg, p);
-                if (cell < 0 && lane == 0) atomicExch(err, ERR_CELL);
-                const T *src = (const T *)a.cache + (cell < 0 ? 0 : cell * a.ldc) + (int64_t)g * head_row;
-                for (int c = lane; c < kp + vp; c += 32) cp16(dst + c * PE, src + c * PE, cell >= 0);
+                const T *src = (const T *)a.cache + (at < 0 ? 0 : at * a.ldc) + (int64_t)g * head_row;
+                for (int c = lane; c < kp + vp; c += 32) cp16(dst + c * PE, src + c * PE, at >= 0);
             } else if (fresh) {
-                const int64_t r = sg[SEG_ROW0] + (p - step0);
-                if (p - step0 >= step_n) {
-                    if (lane == 0) atomicExch(err, ERR_SEGMENT);
-                    for (int c = lane; c < dim + vdim; c += 32) dst[c] = from_f32<T>(0.0f);
-                    continue;
-                }
+                const int64_t r = -1 - at;
+                const int p = step0 + (int)(r - step_row);
                 const float *rope = a.rope + (int64_t)p * a.rot_dims;
-                const int64_t cell = p == pos && hg == 0 ? a.cells[row] : -2;
-                if (cell >= a.n_cells || cell == -1) {
-                    if (lane == 0) atomicExch(err, ERR_CELL);
+                T *keep = nullptr;
+                if (p == pos && hg == 0) {
+                    const int64_t cell = a.cells[row];
+                    if (cell >= 0 && cell < a.n_cells) keep = (T *)a.cache + cell * a.ldc + (int64_t)g * head_row;
+                    else if (lane == 0) atomicExch(err, ERR_CELL);
                 }
-                T *keep = cell >= 0 && cell < a.n_cells ? (T *)a.cache + cell * a.ldc + (int64_t)g * head_row : nullptr;
+#pragma unroll 4
                 for (int c = lane; c < dim + vdim; c += 32) {
                     float x = 0.0f;
                     if (c < a.dim) x = rotated_half(kx + r * a.ldp, rope, a.rot_dims, c);
@@ -199,128 +214,157 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
         }
     };
     const auto commit = []() { asm volatile("cp.async.commit_group;" ::: "memory"); };
-    if (tiles > 0) load_tile(0, true, false);
+    const int64_t found0 = look_up(0), found1 = look_up(1);
+    if (tiles > 0) load_tile(0, found0, true, false);
     commit();
+    if (stages > 1) {
+        if (tiles > 1) load_tile(1, found1, true, false);
+        commit();
+    }
+    int64_t found = stages > 1 ? look_up(2) : found1;   // of the next tile to load
     pdl_wait();
-    if (tiles > 0) load_tile(0, false, true);
+    if (tiles > 0) load_tile(0, found0, false, true);
+    if (stages > 1 && tiles > 1) load_tile(1, found1, false, true);
     {
         const float *q = a.proj + row * a.ldp + (int64_t)(g * rep + h0) * a.dim, *rope = a.rope + (int64_t)pos * a.rot_dims;
-        for (int i = tid; i < HW * dim; i += GT) {
+        for (int i = tid; i < HW * dim; i += (int)blockDim.x) {
             const int h = i / dim, d = i - h * dim;
             sq[i] = h < nh && d < a.dim ? rotated_half(q + (int64_t)h * a.dim, rope, a.rot_dims, d) * a.scale : 0.0f;
         }
     }
-    // value channels: a pair per lane, the entries dealt out over what is left of the threads
-    int lanes = 1;
-    while (lanes < vdim / 2) lanes *= 2;
-    const int subs = GT / lanes, sub = tid / lanes, c0 = 2 * (tid % lanes);
-    float acc[HW][2], m = -INFINITY, l = 0.0f;   // m, l: of head `warp` (warps below HW)
+    __syncthreads();
+    float acc[HW][2 * NP], m[HW], l[HW];   // m: the warp's, l: this lane's share
 #pragma unroll
-    for (int h = 0; h < HW; h++) acc[h][0] = acc[h][1] = 0.0f;
+    for (int h = 0; h < HW; h++) {
+        m[h] = -INFINITY;
+        l[h] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 2 * NP; i++) acc[h][i] = 0.0f;
+    }
+    const int entry = lane >> 1, part = lane & 1;
     for (int t = 0; t < tiles; t++) {
         const int kn = min(GK, e1 - e0 - t * GK);
-        if (stages > 1) {
-            if (t + 1 < tiles) load_tile(t + 1, true, true);
-            commit();
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const T *tile = (const T *)(g_raw + (size_t)(t % stages) * L.tile);
-        {   // scores: P neighbouring lanes share an entry
-            const int h = warp % HW, k = (warp / HW) * (32 / P) + lane / P, part = lane % P;
-            const T *kr = tile + (size_t)k * L.units * PE;
-            const float *qa = sq + h * dim;
-            float s4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll 4
-            for (int p = part; p < kp; p += P) {
+        if (stages > 1) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncwarp();
+        const T *tile = (const T *)(mine + (size_t)(t % stages) * L.tile);
+        float s[HW];
+        {
+            const T *kr = tile + (size_t)entry * L.units * PE;
+#pragma unroll
+            for (int h = 0; h < HW; h++) s[h] = 0.0f;
+#pragma unroll 2
+            for (int p = part; p < kp; p += 2) {
                 float f[PE];
                 Piece<T>::unpack(*reinterpret_cast<const uint4 *>(kr + p * PE), f);
 #pragma unroll
-                for (int e = 0; e < PE; e += 4) {
-                    const float4 x = *reinterpret_cast<const float4 *>(qa + p * PE + e);
-                    s4[0] = fmaf(x.x, f[e], s4[0]);
-                    s4[1] = fmaf(x.y, f[e + 1], s4[1]);
-                    s4[2] = fmaf(x.z, f[e + 2], s4[2]);
-                    s4[3] = fmaf(x.w, f[e + 3], s4[3]);
+                for (int h = 0; h < HW; h++) {
+#pragma unroll
+                    for (int e = 0; e < PE; e += 4) {
+                        const float4 x = *reinterpret_cast<const float4 *>(sq + h * dim + p * PE + e);
+                        s[h] = fmaf(x.x, f[e], s[h]);
+                        s[h] = fmaf(x.y, f[e + 1], s[h]);
+                        s[h] = fmaf(x.z, f[e + 2], s[h]);
+                        s[h] = fmaf(x.w, f[e + 3], s[h]);
+                    }
                 }
             }
-            float s = (s4[0] + s4[1]) + (s4[2] + s4[3]);
-#pragma unroll
-            for (int o = P / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-            if (part == 0) sp[k * HW + h] = k < kn ? s : -INFINITY;
         }
-        __syncthreads();
-        if (warp < HW) {
-            const float s = sp[lane * HW + warp], mn = fmaxf(m, warp_max(s)), corr = m == -INFINITY ? 0.0f : expf(m - mn), p = lane < kn ? expf(s - mn) : 0.0f;
-            l = l * corr + warp_sum(p);
-            m = mn;
-            sp[lane * HW + warp] = p;
-            if (lane == 0) scorr[warp] = corr;
-        }
-        __syncthreads();
-        if (c0 < vdim) {
 #pragma unroll
-            for (int h = 0; h < HW; h++) {
-                const float c = scorr[h];
-                acc[h][0] *= c;
-                acc[h][1] *= c;
-            }
-            const T *vc = tile + dim + c0;
+        for (int h = 0; h < HW; h++) {
+            s[h] += __shfl_xor_sync(0xffffffffu, s[h], 1);
+            const bool in = entry < kn;
+            float mx = in ? s[h] : -INFINITY;
+#pragma unroll
+            for (int o = 2; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float mn = fmaxf(m[h], mx), corr = expf(m[h] - mn), p = in ? expf(s[h] - mn) : 0.0f;   // (a tile has an entry: mn is finite)
+            m[h] = mn;
+            l[h] = l[h] * corr + (part == 0 ? p : 0.0f);
+            if (part == 0) sp[entry * HW + h] = p;
+#pragma unroll
+            for (int i = 0; i < 2 * NP; i++) acc[h][i] *= corr;
+        }
+        __syncwarp();
+        const T *vc = tile + dim + 2 * lane;
 #pragma unroll 4
-            for (int k = sub; k < kn; k += subs) {
-                const float2 v = Piece<T>::pair(vc + (size_t)k * L.units * PE);
+        for (int k = 0; k < kn; k++) {
+            float w[HW];
+            if constexpr (HW % 4 == 0) {
+#pragma unroll
+                for (int h = 0; h < HW; h += 4) *reinterpret_cast<float4 *>(w + h) = *reinterpret_cast<const float4 *>(sp + k * HW + h);
+            } else {
+#pragma unroll
+                for (int h = 0; h < HW; h++) w[h] = sp[k * HW + h];
+            }
+#pragma unroll
+            for (int i = 0; i < NP; i++) {
+                if (2 * lane + 64 * i >= vdim) break;
+                const float2 v = Piece<T>::pair(vc + (size_t)k * L.units * PE + 64 * i);
 #pragma unroll
                 for (int h = 0; h < HW; h++) {
-                    const float p = sp[k * HW + h];
-                    acc[h][0] = fmaf(p, v.x, acc[h][0]);
-                    acc[h][1] = fmaf(p, v.y, acc[h][1]);
+                    acc[h][2 * i] = fmaf(w[h], v.x, acc[h][2 * i]);
+                    acc[h][2 * i + 1] = fmaf(w[h], v.y, acc[h][2 * i + 1]);
                 }
             }
         }
-        __syncthreads();
-        if (stages == 1 && t + 1 < tiles) {
-            load_tile(t + 1, true, true);
-            commit();
-        }
+        __syncwarp();   // the tile and the weights may be overwritten
+        if (t + stages < tiles) load_tile(t + stages, found, true, true);
+        commit();
+        found = look_up(t + stages + 1);
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    if (c0 < vdim) {
+    __syncthreads();
+    // the warps' sums, where the tiles were
+    float *sacc = (float *)g_raw;
 #pragma unroll
-        for (int h = 0; h < HW; h++) *reinterpret_cast<float2 *>(sred + (sub * HW + h) * vdim + c0) = make_float2(acc[h][0], acc[h][1]);
-    }
-    if (warp < HW && lane == 0) {
-        sml[2 * warp] = m;
-        sml[2 * warp + 1] = l;
+    for (int h = 0; h < HW; h++) {
+        l[h] = warp_sum(l[h]);
+#pragma unroll
+        for (int i = 0; i < NP; i++)
+            if (2 * lane + 64 * i < vdim) *reinterpret_cast<float2 *>(sacc + ((size_t)warp * HW + h) * vdim + 2 * lane + 64 * i) = make_float2(acc[h][2 * i], acc[h][2 * i + 1]);
+        if (lane == 0) {
+            sm[warp * HW + h] = m[h];
+            sl[warp * HW + h] = l[h];
+        }
     }
     __syncthreads();
-    for (int i = tid; i < HW * vdim; i += GT) {
+    for (int h = warp; h < HW; h += nw) {   // what each warp counts
+        const float wm = lane < nw ? sm[lane * HW + h] : -INFINITY, mx = warp_max(wm), w = wm == -INFINITY ? 0.0f : expf(wm - mx);
+        const float sum = warp_sum(lane < nw ? sl[lane * HW + h] * w : 0.0f);
+        if (lane < nw) sw[lane * HW + h] = w;
+        if (lane == 0) {
+            sml[2 * h] = mx;
+            sml[2 * h + 1] = sum;
+        }
+    }
+    __syncthreads();
+    for (int i = tid; i < HW * vdim; i += (int)blockDim.x) {
+        const int h = i / vdim;
         float v = 0.0f;
-        for (int s = 0; s < subs; s++) v += sred[s * HW * vdim + i];
+#pragma unroll 8
+        for (int k = 0; k < nw; k++) v = fmaf(sacc[(size_t)k * HW * vdim + i], sw[k * HW + h], v);
         sout[i] = v;
     }
     const int blocks = (int)cluster.num_blocks();
     cluster.sync();
-    if (tid < HW) {   // what each block's sums count, the sink in the denominator
-        const float sink = a.sink && tid < nh ? a.sink[g * rep + h0 + tid] : -INFINITY;
-        float mx = sink;
-        for (int b = 0; b < blocks; b++) mx = fmaxf(mx, cluster.map_shared_rank(sml, b)[2 * tid]);
-        float den = expf(sink - mx);
-        for (int b = 0; b < blocks; b++) {
-            const float *o = cluster.map_shared_rank(sml, b);
-            const float w = o[2 * tid] == -INFINITY ? 0.0f : expf(o[2 * tid] - mx);
-            sw[b * HW + tid] = w;
-            den = fmaf(o[2 * tid + 1], w, den);
-        }
-        for (int b = 0; b < blocks; b++) sw[b * HW + tid] /= den;
+    for (int h = warp; h < HW; h += nw) {   // what each block counts, the sink in the denominator
+        const float sink = a.sink && h < nh ? a.sink[g * rep + h0 + h] : -INFINITY;
+        float2 ml = make_float2(-INFINITY, 0.0f);
+        if (lane < blocks) ml = *reinterpret_cast<const float2 *>(cluster.map_shared_rank(sml, lane) + 2 * h);
+        const float mx = fmaxf(sink, warp_max(ml.x)), w = ml.x == -INFINITY ? 0.0f : expf(ml.x - mx);
+        const float den = warp_sum(ml.y * w) + expf(sink - mx);
+        if (lane < blocks) sw[lane * HW + h] = w / den;
     }
     __syncthreads();
-    for (int i = (int)cluster.block_rank() * GT + tid; i < nh * vdim; i += blocks * GT) {
+    for (int i = (int)cluster.block_rank() * (int)blockDim.x + tid; i < nh * vdim; i += blocks * (int)blockDim.x) {
         const int h = i / vdim, c = i - h * vdim;
         if (c >= a.vdim) continue;
-        float v = 0.0f;
-        for (int b = 0; b < blocks; b++) v = fmaf(cluster.map_shared_rank(sout, b)[i], sw[b * HW + h], v);
+        float part_of[SPLITS_MAX], v = 0.0f;
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++) part_of[b] = b < blocks ? cluster.map_shared_rank(sout, b)[i] : 0.0f;
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++)
+            if (b < blocks) v = fmaf(part_of[b], sw[b * HW + h], v);
         const int64_t at = row * a.ldy + (int64_t)(g * rep + h0 + h) * a.vdim + c;
         if (a.y_type == B200_TYPE_F32) ((float *)a.y)[at] = v;
         else ((__nv_bfloat16 *)a.y)[at] = __float2bfloat16_rn(v);
@@ -613,21 +657,35 @@ int allow_smem(K kernel, size_t smem) {
 }
 constexpr size_t SMEM_MAX = 220 * 1024;
 
-template <typename T, int HW>
+// warps and tiles per warp that fit: eight warps with two tiles if possible; 0 warps: none do
+DecodeSmem decode_plan(const GroupedArgs &a, int es, int hw, int *warps, int *stages) {
+    for (*warps = GT / 32; *warps >= 1; *warps /= 2)
+        for (*stages = 2; *stages >= 1; --*stages) {
+            const DecodeSmem L(a.dim, a.vdim, es, hw, *warps, *stages);
+            if (L.bytes() <= SMEM_MAX) return L;
+        }
+    *warps = 0;
+    return DecodeSmem(1, 1, es, hw, 1, 1);
+}
+template <typename T, int HW, int NP>
 int run_decode(const GroupedArgs &a, int *err, cudaStream_t s) {
-    const DecodeSmem L(a.dim, a.vdim, (int)sizeof(T), HW);
+    int warps = 0, stages = 0;
+    const DecodeSmem L = decode_plan(a, (int)sizeof(T), HW, &warps, &stages);
+    B200_REQUIRE(warps > 0, "grouped decode: head size too large");
     const int rep = a.heads / a.kv_heads, hg = (rep + GH - 1) / GH;
-    const int stages = 2 * (size_t)L.tile + (size_t)L.floats * 4 <= SMEM_MAX ? 2 : 1;
-    const size_t smem = (size_t)stages * L.tile + (size_t)L.floats * 4;
-    int rc = allow_smem(grouped_decode_kernel<T, HW>, smem);
+    int rc = allow_smem(grouped_decode_kernel<T, HW, NP>, L.bytes());
     if (rc != B200_STATUS_SUCCESS) return rc;
-    return launch_pdl_cluster(grouped_decode_kernel<T, HW>, dim3((unsigned)a.splits, (unsigned)(a.kv_heads * hg), (unsigned)a.n), dim3(GT), (unsigned)a.splits, smem, s, a, hg,
-                              stages, err);
+    return launch_pdl_cluster(grouped_decode_kernel<T, HW, NP>, dim3((unsigned)a.splits, (unsigned)(a.kv_heads * hg), (unsigned)a.n), dim3((unsigned)(32 * warps)),
+                              (unsigned)a.splits, L.bytes(), s, a, hg, stages, err);
+}
+template <typename T, int HW>
+int run_decode_channels(const GroupedArgs &a, int *err, cudaStream_t s) {
+    return a.vdim <= 64 ? run_decode<T, HW, 1>(a, err, s) : a.vdim <= 128 ? run_decode<T, HW, 2>(a, err, s) : run_decode<T, HW, 4>(a, err, s);
 }
 template <typename T>
 int run_decode_heads(const GroupedArgs &a, int *err, cudaStream_t s) {
     const int rep = a.heads / a.kv_heads;
-    return rep > 4 ? run_decode<T, 8>(a, err, s) : rep > 2 ? run_decode<T, 4>(a, err, s) : rep > 1 ? run_decode<T, 2>(a, err, s) : run_decode<T, 1>(a, err, s);
+    return rep > 4 ? run_decode_channels<T, 8>(a, err, s) : rep > 2 ? run_decode_channels<T, 4>(a, err, s) : rep > 1 ? run_decode_channels<T, 2>(a, err, s) : run_decode_channels<T, 1>(a, err, s);
 }
 template <typename T, typename Y>
 int run_any(const GroupedArgs &a, int *err, cudaStream_t s) {
@@ -679,10 +737,10 @@ int launch_grouped_decode(const GroupedArgs &a, cudaStream_t s) {
     int *err = nullptr;
     int rc = check(a, &err);
     if (rc != B200_STATUS_SUCCESS || a.n == 0) return rc;
-    B200_REQUIRE(a.cells && a.seg && a.row_seg && a.tab && a.y && a.n_seg > 0 && a.splits >= 1 && a.splits <= 8, "grouped decode: bad operand");
-    const int es = a.type == B200_TYPE_F32 ? 4 : 2;
-    const DecodeSmem L(a.dim, a.vdim, es, GH);
-    if (a.vdim > 2 * GT || (size_t)L.tile + (size_t)L.floats * 4 > SMEM_MAX) {   // heads a block cannot hold
+    B200_REQUIRE(a.cells && a.seg && a.row_seg && a.tab && a.y && a.n_seg > 0 && a.splits >= 1 && a.splits <= SPLITS_MAX, "grouped decode: bad operand");
+    int warps = 0, stages = 0;
+    decode_plan(a, a.type == B200_TYPE_F32 ? 4 : 2, GH, &warps, &stages);
+    if (a.vdim > 256 || warps == 0) {   // heads a block cannot hold
         rc = launch_grouped_store(a, s);
         return rc != B200_STATUS_SUCCESS ? rc : launch_grouped_attn(a, s);
     }
