@@ -5,9 +5,9 @@
 //
 // What a row sees is walked as a list of entries: its kept first positions, then the window's.  An entry's position leads to a cell
 // through the segment's part of `tab` (KEPT first positions, then the positions from KEY0 on).
-//   grouped_decode_kernel     few rows per sequence: a cluster per (row, key head, up to 8 query heads), its blocks share the entries and
-//                             merge through distributed shared memory.  Positions of this step come from proj (and the row's own is
-//                             stored in its cell on the way), earlier ones from the cells
+//   grouped_decode_mma_kernel, grouped_decode_kernel   few rows per sequence, BF16 and F32 cells: a cluster per (row, key head, up to 8
+//                             query heads), its blocks share the entries and merge through distributed shared memory.  Positions of this
+//                             step come from proj (and the row's own is stored in its cell on the way), earlier ones from the cells
 //   grouped_store_kernel      keys and values of a prompt's rows into their cells, then
 //   grouped_attn_mma_kernel   64 rows x 64-entry tiles on mma.sync (BF16 operands, F32 scores and sums; a weight goes in as two BF16
 //                             parts, so that it keeps its 32-bit value to 2^-17), or
@@ -22,9 +22,10 @@ namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr int GT = 256;            // threads per block, at most
+constexpr int GT = 256;            // threads per block
 constexpr int GK = 16;             // entries per tile of a warp of the few-rows kernel
 constexpr int GH = 8;              // query heads per block of it
+__host__ __device__ constexpr int decode_threads(int hw, int np) { return hw * np >= 16 ? 256 : 512; }   // of that kernel, at most
 constexpr int SPLITS_MAX = 8;      // blocks that share a row's entries
 
 __host__ __device__ inline int pad8(int n) { return (n + 7) / 8 * 8; }
@@ -128,17 +129,47 @@ struct DecodeSmem {
         m = p + nw * GK * hw;
         l = m + nw * hw;
         w = l + nw * hw;
-        out = (w + 8 * hw + 3) / 4 * 4;
+        out = (w + (nw > 8 ? nw : 8) * hw + 3) / 4 * 4;
         ml = out + hw * e;
         floats = ml + 2 * hw;
     }
     __host__ __device__ size_t bytes() const { return tiles + (size_t)floats * 4; }
 };
 
+// keys and values of a row of this step, as its cell holds them, into `dst` (a warp; values `gap` elements further on) and, if given, into
+// the cell
+template <typename T>
+__device__ __noinline__ void fresh_row(const float *k, const float *v, const float *rope, int rot_dims, int dim, int vdim, T *dst, int gap, T *keep) {
+    constexpr int U = 8;
+    const int d = pad8(dim), n = d + pad8(vdim), half = rot_dims >> 1;
+    for (int c0 = threadIdx.x & 31; c0 < n; c0 += 32 * U) {
+        float x[U], y[U], cs[U], sn[U];
+#pragma unroll
+        for (int u = 0; u < U; u++) {   // all the loads, then the stores
+            const int c = c0 + 32 * u;
+            const bool turns = c < rot_dims, low = c < half;
+            const float *at = c < dim ? k + c : c >= d && c - d < vdim ? v + (c - d) : k, *other = turns ? (low ? at + half : at - half) : at;
+            const float *turn = turns ? rope + 2 * (low ? c : c - half) : at;
+            x[u] = *at;
+            y[u] = *other;
+            cs[u] = turns ? turn[0] : 1.0f;
+            sn[u] = turns ? (low ? -turn[1] : turn[1]) : 0.0f;
+        }
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+            const int c = c0 + 32 * u;
+            if (c >= n) break;
+            const T r = from_f32<T>(c < dim || (c >= d && c - d < vdim) ? (c < rot_dims ? fmaf(x[u], cs[u], y[u] * sn[u]) : x[u]) : 0.0f);
+            dst[c < d ? c : c + gap] = r;
+            if (keep) keep[c] = r;
+        }
+    }
+}
+
 // A warp owns a stretch of the entries from load to weighted sum (no barrier until the end): two lanes share an entry's scores, then a
 // lane owns NP pairs of value channels.
 template <typename T, int HW, int NP>
-__global__ void __launch_bounds__(GT, 1)
+__global__ void __launch_bounds__(decode_threads(HW, NP), 1)
 grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
     constexpr int PE = Piece<T>::E;
     extern __shared__ __align__(16) uint8_t g_raw[];
@@ -166,65 +197,49 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
     const int head_row = dim + vdim;
     const float *kx = a.proj + (int64_t)a.heads * a.dim + (int64_t)g * a.dim, *vx = a.proj + (int64_t)(a.heads + a.kv_heads) * a.dim + (int64_t)g * a.vdim;
     uint8_t *mine = g_raw + (size_t)warp * stages * L.tile;
-    // what stands behind entry lane % GK of tile t: a cell, -1 - r for row r of this step, NOTHING past the last or when the lists lack it
-    constexpr int64_t NOTHING = INT64_MIN;
-    const auto look_up = [&](int t) -> int64_t {
+    // what stands behind entry lane % GK of tile t: a cell, -2 - r for row r of this step, -1 past the last entry
+    const auto look_up = [&](int t) -> int {
         const int e = e0 + t * GK + lane % GK;
-        if (e >= e1) return NOTHING;
+        if (e >= e1) return -1;
         const int p = en.position(e);
-        if (p >= step0) {
-            if (p - step0 < step_n) return -1 - (int64_t)(step_row + (p - step0));
-            atomicExch(err, ERR_SEGMENT);
-            return NOTHING;
-        }
-        const int64_t cell = cell_of(a, sg, p);
+        if (p >= step0 && p - step0 < step_n) return -2 - (step_row + (p - step0));
+        const int64_t cell = p < step0 ? cell_of(a, sg, p) : -1;
         if (cell < 0) atomicExch(err, ERR_CELL);
-        return cell < 0 ? NOTHING : cell;
+        return cell < 0 ? 0 : (int)cell;
     };
-    // an entry's row: key channels, then value channels.  cells: those of earlier steps (what is missing is zero), fresh: this step's
-    const auto load_tile = [&](int t, int64_t found, bool cells, bool fresh) {
-        T *dst0 = (T *)(mine + (size_t)(t % stages) * L.tile);
+    // an entry's row: key channels, then value channels.  First what cells hold, then this step's own rows
+    const T *cache = (const T *)a.cache + (int64_t)g * head_row;
+    const auto load_cells = [&](int t, int found) {
+        const int kn = min(GK, e1 - e0 - t * GK);
+        T *dst = (T *)(mine + (size_t)(t % stages) * L.tile) + lane * PE;
 #pragma unroll 4
-        for (int k = 0; k < GK; k++) {
-            const int64_t at = __shfl_sync(0xffffffffu, found, k);
-            T *dst = dst0 + (size_t)k * L.units * PE;
-            if (at >= 0 || at == NOTHING) {
-                if (!cells) continue;
-                const T *src = (const T *)a.cache + (at < 0 ? 0 : at * a.ldc) + (int64_t)g * head_row;
-                for (int c = lane; c < kp + vp; c += 32) cp16(dst + c * PE, src + c * PE, at >= 0);
-            } else if (fresh) {
-                const int64_t r = -1 - at;
-                const int p = step0 + (int)(r - step_row);
-                const float *rope = a.rope + (int64_t)p * a.rot_dims;
-                T *keep = nullptr;
-                if (p == pos && hg == 0) {
-                    const int64_t cell = a.cells[row];
-                    if (cell >= 0 && cell < a.n_cells) keep = (T *)a.cache + cell * a.ldc + (int64_t)g * head_row;
-                    else if (lane == 0) atomicExch(err, ERR_CELL);
-                }
-#pragma unroll 4
-                for (int c = lane; c < dim + vdim; c += 32) {
-                    float x = 0.0f;
-                    if (c < a.dim) x = rotated_half(kx + r * a.ldp, rope, a.rot_dims, c);
-                    else if (c >= dim && c - dim < a.vdim) x = vx[r * a.ldp + c - dim];
-                    dst[c] = from_f32<T>(x);
-                    if (keep) keep[c] = from_f32<T>(x);
-                }
-            }
+        for (int k = 0; k < kn; k++, dst += L.units * PE) {
+            const int at = __shfl_sync(0xffffffffu, found, k);
+            const T *src = cache + (int64_t)at * a.ldc;
+            if (at >= 0)
+                for (int c = lane; c < kp + vp; c += 32) cp16(dst + (c - lane) * PE, src + c * PE, true);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const auto load_fresh = [&](int t, int found) {
+        for (uint32_t todo = __ballot_sync(0xffffffffu, lane < GK && found < -1); todo; todo &= todo - 1) {
+            const int k = __ffs(todo) - 1;
+            const int64_t r = -2 - __shfl_sync(0xffffffffu, found, k);
+            const int32_t *cell = hg == 0 && r == row ? a.cells + row : nullptr;
+            T *keep = nullptr;
+            if (cell && *cell >= 0 && *cell < a.n_cells) keep = (T *)a.cache + (int64_t)*cell * a.ldc + (int64_t)g * head_row;
+            else if (cell && lane == 0) atomicExch(err, ERR_CELL);
+            fresh_row<T>(kx + r * a.ldp, vx + r * a.ldp, a.rope + (int64_t)(step0 + (int)(r - step_row)) * a.rot_dims, a.rot_dims, a.dim, a.vdim,
+                         (T *)(mine + (size_t)(t % stages) * L.tile) + (size_t)k * L.units * PE, 0, keep);
         }
     };
-    const auto commit = []() { asm volatile("cp.async.commit_group;" ::: "memory"); };
-    const int64_t found0 = look_up(0), found1 = look_up(1);
-    if (tiles > 0) load_tile(0, found0, true, false);
-    commit();
-    if (stages > 1) {
-        if (tiles > 1) load_tile(1, found1, true, false);
-        commit();
-    }
-    int64_t found = stages > 1 ? look_up(2) : found1;   // of the next tile to load
+    const int found0 = look_up(0), found1 = tiles > 1 ? look_up(1) : -1;
+    load_cells(0, found0);
+    if (stages > 1) load_cells(1, found1);
+    int found = stages > 1 && tiles > 2 ? look_up(2) : found1;   // of the next tile to load
     pdl_wait();
-    if (tiles > 0) load_tile(0, found0, false, true);
-    if (stages > 1 && tiles > 1) load_tile(1, found1, false, true);
+    load_fresh(0, found0);
+    if (stages > 1) load_fresh(1, found1);
     {
         const float *q = a.proj + row * a.ldp + (int64_t)(g * rep + h0) * a.dim, *rope = a.rope + (int64_t)pos * a.rot_dims;
         for (int i = tid; i < HW * dim; i += (int)blockDim.x) {
@@ -308,9 +323,11 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
             }
         }
         __syncwarp();   // the tile and the weights may be overwritten
-        if (t + stages < tiles) load_tile(t + stages, found, true, true);
-        commit();
-        found = look_up(t + stages + 1);
+        load_cells(t + stages, found);
+        if (t + stages < tiles) {
+            load_fresh(t + stages, found);
+            found = look_up(t + stages + 1);
+        }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
@@ -341,7 +358,7 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
     for (int i = tid; i < HW * vdim; i += (int)blockDim.x) {
         const int h = i / vdim;
         float v = 0.0f;
-#pragma unroll 8
+#pragma unroll 4
         for (int k = 0; k < nw; k++) v = fmaf(sacc[(size_t)k * HW * vdim + i], sw[k * HW + h], v);
         sout[i] = v;
     }
@@ -370,6 +387,295 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
         else ((__nv_bfloat16 *)a.y)[at] = __float2bfloat16_rn(v);
     }
     cluster.sync();   // nobody leaves before everyone has read
+}
+
+// The same over BF16 cells on the tensor cores: a warp's tile of 16 entries meets up to 8 heads' queries in m16n8k16 products whose 16 rows
+// are the heads' high BF16 parts and the remainders (their sum keeps 16 bits of the query), then the weights, high parts and remainders
+// likewise, meet the values.  A block pushes its sums to the block of the cluster that owns them.
+constexpr int DW = 8;   // warps of a block, at most
+struct DecodeMmaSmem {
+    int kq, vq, units, tile;                  // channels of a key and a value in an entry's row, its 16-byte units, bytes of a tile
+    int q, m, l, w, recv, recv_ml, bytes;     // byte offsets
+    __host__ __device__ DecodeMmaSmem(int dim, int vdim, int nw, int stages) {
+        kq = (dim + 15) / 16 * 16;
+        vq = (vdim + 15) / 16 * 16;
+        units = (kq + vq) / 8 + 1;            // odd: eight rows of a matrix in different banks
+        tile = GK * units * 16;
+        q = nw * stages * tile;               // (the warps' sums take the tiles' place)
+        m = q + 16 * (kq + 8) * 2;
+        l = m + nw * GH * 4;
+        w = l + nw * GH * 4;
+        recv = w + SPLITS_MAX * GH * 4;
+        recv_ml = recv + (GH * vq + SPLITS_MAX) * 4;
+        bytes = recv_ml + SPLITS_MAX * GH * 8;
+    }
+};
+__device__ __forceinline__ void cluster_arrive_relaxed() { asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
+// a bulk copy whose bytes count at the barrier, and the wait for them, bounded (a second time if the first ran out: the copies may still
+// be on their way); false when it ran out
+constexpr int ERR_BULK = 4;
+constexpr uint32_t BULK_WAIT_LIMIT = 1u << 20;
+__device__ __forceinline__ void bulk_copy(void *dst, const void *src, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes), "r"(bar)
+                 : "memory");
+}
+__device__ __forceinline__ bool bulk_wait(uint32_t bar, uint32_t parity) {
+    for (int round = 0; round < 2; round++)
+        for (uint32_t it = 0; it < BULK_WAIT_LIMIT; it++) {
+            uint32_t ok;
+            asm volatile("{ .reg .pred p; mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
+            if (ok) return round == 0;
+        }
+    return false;
+}
+
+template <int NT>   // pairs of value channel groups of 8: 16 NT channels at most
+__global__ void __launch_bounds__(32 * DW, 1)
+grouped_decode_mma_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
+    typedef __nv_bfloat16 bf;
+    extern __shared__ __align__(16) uint8_t g_raw[];
+    __shared__ uint64_t bars[DW][2];   // a warp's tiles
+    cg::cluster_group cluster = cg::this_cluster();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5, blocks = (int)gridDim.x;
+    const int dim = pad8(a.dim), vdim = pad8(a.vdim), kp = dim / 8, vp = vdim / 8;
+    const DecodeMmaSmem L(a.dim, a.vdim, nw, stages);
+    bf *sQ = (bf *)(g_raw + L.q);
+    float *sm = (float *)(g_raw + L.m), *sl = (float *)(g_raw + L.l), *sw = (float *)(g_raw + L.w), *recv = (float *)(g_raw + L.recv);
+    float2 *recv_ml = (float2 *)(g_raw + L.recv_ml);
+    const int rep = a.heads / a.kv_heads, g = blockIdx.y / head_groups, hg = blockIdx.y % head_groups, h0 = hg * GH, nh = min(GH, rep - h0);
+    const int64_t row = blockIdx.z;
+    const int KS = L.units * 8, QS = L.kq + 8;   // strides of an entry's and a query's row in elements
+    pdl_trigger();
+    // the step's inputs and the cells of earlier steps are in place before its first kernel starts
+    const int pos = a.pos[row], si = a.row_seg[row];
+    const bool seg_ok = segment_ok(a, si), pos_ok = pos >= 0 && (a.rot_dims == 0 || pos < a.rope_rows);
+    if (!seg_ok || !pos_ok) {   // (the same for every block of the cluster)
+        if (tid == 0) atomicExch(err, seg_ok ? ERR_POS : ERR_SEGMENT);
+        return;
+    }
+    cluster_arrive_relaxed();   // waited for before anything goes to another block
+    const int32_t *sg = a.seg + (int64_t)si * SEG_FIELDS;
+    const int step0 = sg[SEG_POS0], step_n = sg[SEG_ROWS], step_row = sg[SEG_ROW0];
+    const Entries en(a, pos, pos);
+    const int owners = blocks * nw, per = (en.total + owners - 1) / owners;
+    const int e0 = min(en.total, ((int)blockIdx.x * nw + warp) * per), e1 = min(en.total, e0 + per), tiles = (e1 - e0 + GK - 1) / GK;
+    const int head_row = dim + vdim;
+    bf *mine = (bf *)(g_raw + (size_t)warp * stages * L.tile);
+    const bf *cache = (const bf *)a.cache + (int64_t)g * head_row;
+    // what stands behind entry lane % GK of tile t: a cell, -2 - r for row r of this step, -1 past the last entry
+    const auto look_up = [&](int t) -> int {
+        const int e = e0 + t * GK + lane % GK;
+        if (e >= e1) return -1;
+        const int p = en.position(e);
+        if (p >= step0 && p - step0 < step_n) return -2 - (step_row + (p - step0));
+        const int64_t cell = p < step0 ? cell_of(a, sg, p) : -1;
+        if (cell < 0) atomicExch(err, ERR_CELL);
+        return cell < 0 ? 0 : (int)cell;
+    };
+    // bulk copies by the entry's lane; values past the last entry are zero
+    const auto load_cells = [&](int t, int found) {
+        if (t >= tiles) return;
+        bf *dst = mine + (size_t)(t % stages) * (L.tile / 2);
+        const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&bars[warp][t % stages]);
+        const uint32_t cells = __ballot_sync(0xffffffffu, lane < GK && found >= 0);
+        if (lane == 0)
+            asm volatile("{ .reg .b64 st; mbarrier.arrive.expect_tx.shared::cta.b64 st, [%0], %1; }" ::"r"(bar), "r"((uint32_t)__popc(cells) * (uint32_t)head_row * 2) : "memory");
+        __syncwarp();
+        if (lane < GK && found >= 0) {
+            const bf *src = cache + (int64_t)found * a.ldc;
+            if (L.kq == dim) {
+                bulk_copy(dst + lane * KS, src, (uint32_t)head_row * 2, bar);
+            } else {
+                bulk_copy(dst + lane * KS, src, (uint32_t)dim * 2, bar);
+                bulk_copy(dst + lane * KS + L.kq, src + dim, (uint32_t)vdim * 2, bar);
+            }
+        }
+        const int kn = e1 - e0 - t * GK;   // (their scores are masked, so the keys need not be)
+        for (int k = kn + (lane >> 3); k < GK; k += 4)
+            for (int c = lane & 7; c < L.vq / 8; c += 8) *reinterpret_cast<uint4 *>(dst + k * KS + L.kq + 8 * c) = make_uint4(0, 0, 0, 0);
+    };
+    const auto load_fresh = [&](int t, int found) {
+        for (uint32_t todo = __ballot_sync(0xffffffffu, lane < GK && found < -1); todo; todo &= todo - 1) {
+            const int k = __ffs(todo) - 1;
+            const int64_t r = -2 - __shfl_sync(0xffffffffu, found, k);
+            const int32_t *cell = hg == 0 && r == row ? a.cells + row : nullptr;
+            bf *keep = nullptr;
+            if (cell && *cell >= 0 && *cell < a.n_cells) keep = (bf *)a.cache + (int64_t)*cell * a.ldc + (int64_t)g * head_row;
+            else if (cell && lane == 0) atomicExch(err, ERR_CELL);
+            const float *x = a.proj + r * a.ldp + (int64_t)a.heads * a.dim;
+            fresh_row<bf>(x + g * a.dim, x + (int64_t)a.kv_heads * a.dim + (int64_t)g * a.vdim, a.rope + (int64_t)(step0 + (int)(r - step_row)) * a.rot_dims, a.rot_dims, a.dim, a.vdim,
+                          mine + (size_t)(t % stages) * (L.tile / 2) + k * KS, L.kq - dim, keep);
+        }
+    };
+    if (lane == 0) {
+        for (int i = 0; i < stages; i++) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"((uint32_t)__cvta_generic_to_shared(&bars[warp][i])) : "memory");
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncwarp();
+    const int found0 = look_up(0), found1 = tiles > 1 ? look_up(1) : -1;
+    load_cells(0, found0);
+    if (stages > 1) load_cells(1, found1);
+    int found = stages > 1 && tiles > 2 ? look_up(2) : found1;   // of the next tile to load
+    // channels between a head's and the next multiple of 16 stay zero
+    if (L.kq != dim || L.vq != vdim)
+        for (int i = lane; i < stages * GK * 2; i += 32) {
+            bf *r = mine + (i >> 1) * KS;
+            if (!(i & 1) && L.kq != dim) *reinterpret_cast<uint4 *>(r + dim) = make_uint4(0, 0, 0, 0);
+            if ((i & 1) && L.vq != vdim) *reinterpret_cast<uint4 *>(r + L.kq + vdim) = make_uint4(0, 0, 0, 0);
+        }
+    pdl_wait();
+    if (tiles > 0) load_fresh(0, found0);
+    if (stages > 1 && tiles > 1) load_fresh(1, found1);
+    {   // queries in powers of two: high parts in rows 0 .. 7, remainders in rows 8 .. 15
+        const float *q = a.proj + row * a.ldp + (int64_t)(g * rep + h0) * a.dim, *rope = a.rope + (int64_t)pos * a.rot_dims;
+        for (int h = warp; h < GH; h += nw)
+            for (int d = lane; d < L.kq; d += 32) {
+                const float x = h < nh && d < a.dim ? rotated_half(q + (int64_t)h * a.dim, rope, a.rot_dims, d) * (a.scale * 1.4426950408889634f) : 0.0f;
+                const bf hi = __float2bfloat16_rn(x);
+                sQ[h * QS + d] = hi;
+                sQ[(h + 8) * QS + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
+            }
+    }
+    __syncthreads();
+    // this lane's head is lane / 4; of a product's 8 columns it has two, high parts and remainders
+    float acc[2 * NT][4], m = -INFINITY, l = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 2 * NT; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    const bf *qp = sQ + (lane & 15) * QS + (lane >> 4) * 8;
+    const int koff = ((lane >> 4) * 8 + (lane & 7)) * KS + ((lane >> 3) & 1) * 8, voff = (((lane >> 3) & 1) * 8 + (lane & 7)) * KS + (lane >> 4) * 8 + L.kq;
+    for (int t = 0; t < tiles; t++) {
+        const int kn = e1 - e0 - t * GK;
+        if (!bulk_wait((uint32_t)__cvta_generic_to_shared(&bars[warp][t % stages]), (uint32_t)(t / stages) & 1u) && lane == 0) atomicExch(err, ERR_BULK);
+        __syncwarp();
+        const bf *tile = mine + (size_t)(t % stages) * (L.tile / 2);
+        float c0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll 4
+        for (int d = 0; d < L.kq; d += 16) {
+            uint32_t qa[4], kb[4];
+            ldsm4(qa, qp + d);
+            ldsm4(kb, tile + koff + d);
+            mma_bf16(c0, qa, kb[0], kb[1]);
+            mma_bf16(c1, qa, kb[2], kb[3]);
+        }
+        const int e = 2 * (lane & 3);
+        float s[4] = {c0[0] + c0[2], c0[1] + c0[3], c1[0] + c1[2], c1[1] + c1[3]};
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+            if (e + (i & 1) + 8 * (i >> 1) >= kn) s[i] = -INFINITY;
+        float mx = fmaxf(fmaxf(s[0], s[1]), fmaxf(s[2], s[3]));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float mn = fmaxf(m, mx), corr = exp2f(m - mn);   // (a tile has an entry: mn is finite)
+        m = mn;
+        float p[4];
+        uint32_t pa[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) p[i] = exp2f(s[i] - mn);
+        l = l * corr + ((p[0] + p[1]) + (p[2] + p[3]));
+        pa[0] = bf16_pack(p[0], p[1]);
+        pa[1] = bf16_pack(p[0] - bf16_lo(pa[0]), p[1] - bf16_hi(pa[0]));
+        pa[2] = bf16_pack(p[2], p[3]);
+        pa[3] = bf16_pack(p[2] - bf16_lo(pa[2]), p[3] - bf16_hi(pa[2]));
+        if (__any_sync(0xffffffffu, corr != 1.0f)) {
+#pragma unroll
+            for (int i = 0; i < 2 * NT; i++) {
+                acc[i][0] *= corr;
+                acc[i][1] *= corr;
+                acc[i][2] *= corr;
+                acc[i][3] *= corr;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NT; i++) {
+            uint32_t vb[4];   // (channels past vq: what stands behind the row, in columns that nobody reads)
+            ldsm4_t(vb, tile + voff + 16 * i);
+            mma_bf16(acc[2 * i], pa, vb[0], vb[1]);
+            mma_bf16(acc[2 * i + 1], pa, vb[2], vb[3]);
+        }
+        __syncwarp();   // the tile may be overwritten
+        load_cells(t + stages, found);
+        if (t + stages < tiles) {
+            load_fresh(t + stages, found);
+            found = look_up(t + stages + 1);
+        }
+    }
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    if ((lane & 3) == 0) {
+        sm[warp * GH + (lane >> 2)] = m;
+        sl[warp * GH + (lane >> 2)] = l;
+    }
+    __syncthreads();
+    // the warps' sums, where the tiles were, each counted as its maximum asks for
+    float *sacc = (float *)g_raw;
+    {
+        const int h = lane >> 2;
+        float mw[DW], mb = -INFINITY, lb = 0.0f;
+#pragma unroll
+        for (int k = 0; k < DW; k++) {
+            mw[k] = k < nw ? sm[k * GH + h] : -INFINITY;
+            mb = fmaxf(mb, mw[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < DW; k++)
+            if (mw[k] != -INFINITY) lb = fmaf(sl[k * GH + h], exp2f(mw[k] - mb), lb);
+        const float w = m == -INFINITY ? 0.0f : exp2f(m - mb);
+        float *o = sacc + ((size_t)warp * GH + h) * L.vq + 2 * (lane & 3);
+#pragma unroll
+        for (int i = 0; i < 2 * NT; i++)
+            if (8 * i < L.vq) *reinterpret_cast<float2 *>(o + 8 * i) = make_float2((acc[i][0] + acc[i][2]) * w, (acc[i][1] + acc[i][3]) * w);
+        cluster_wait();   // every block of the cluster has started
+        for (int b = warp; b < blocks; b += nw)
+            if ((lane & 3) == 0) cluster.map_shared_rank(recv_ml, b)[(int)blockIdx.x * GH + h] = make_float2(mb, lb);
+    }
+    __syncthreads();
+    // block b owns elements b own .. of the heads' channels
+    const int total = nh * L.vq, own = (total + blocks - 1) / blocks;
+    for (int i = tid; i < total; i += (int)blockDim.x) {
+        float v = 0.0f;
+#pragma unroll
+        for (int k = 0; k < DW; k++)
+            if (k < nw) v += sacc[(size_t)k * GH * L.vq + i];
+        const int b = i / own;
+        cluster.map_shared_rank(recv, b)[(int)blockIdx.x * own + i - b * own] = v;
+    }
+    cluster_arrive();
+    cluster_wait();
+    if (warp == 0 && lane < GH) {   // what each block counts, the sink in the denominator
+        const float sink = a.sink && lane < nh ? a.sink[g * rep + h0 + lane] * 1.4426950408889634f : -INFINITY;
+        float2 ml[SPLITS_MAX];
+        float mx = sink, w[SPLITS_MAX];
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++) {
+            ml[b] = b < blocks ? recv_ml[b * GH + lane] : make_float2(-INFINITY, 0.0f);
+            mx = fmaxf(mx, ml[b].x);
+        }
+        float den = exp2f(sink - mx);
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++) {
+            w[b] = ml[b].x == -INFINITY ? 0.0f : exp2f(ml[b].x - mx);
+            den = fmaf(ml[b].y, w[b], den);
+        }
+        den = 1.0f / den;
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++)
+            if (b < blocks) sw[b * GH + lane] = w[b] * den;
+    }
+    __syncthreads();
+    for (int j = tid; j < own; j += (int)blockDim.x) {
+        const int i = (int)blockIdx.x * own + j, h = i / L.vq, c = i - h * L.vq;
+        if (i >= total || c >= a.vdim) continue;
+        float v = 0.0f;
+#pragma unroll
+        for (int b = 0; b < SPLITS_MAX; b++)
+            if (b < blocks) v = fmaf(recv[b * own + j], sw[b * GH + h], v);
+        const int64_t at = row * a.ldy + (int64_t)(g * rep + h0 + h) * a.vdim + c;
+        if (a.y_type == B200_TYPE_F32) ((float *)a.y)[at] = v;
+        else ((bf *)a.y)[at] = __float2bfloat16_rn(v);
+    }
 }
 
 // ---- many rows -------------------------------------------------------------------------------------------------
@@ -657,9 +963,9 @@ int allow_smem(K kernel, size_t smem) {
 }
 constexpr size_t SMEM_MAX = 220 * 1024;
 
-// warps and tiles per warp that fit: eight warps with two tiles if possible; 0 warps: none do
-DecodeSmem decode_plan(const GroupedArgs &a, int es, int hw, int *warps, int *stages) {
-    for (*warps = GT / 32; *warps >= 1; *warps /= 2)
+// warps and tiles per warp that fit, as many warps as possible; 0 warps: none do
+DecodeSmem decode_plan(const GroupedArgs &a, int es, int hw, int threads, int *warps, int *stages) {
+    for (*warps = threads / 32; *warps >= 1; *warps /= 2)
         for (*stages = 2; *stages >= 1; --*stages) {
             const DecodeSmem L(a.dim, a.vdim, es, hw, *warps, *stages);
             if (L.bytes() <= SMEM_MAX) return L;
@@ -670,7 +976,7 @@ DecodeSmem decode_plan(const GroupedArgs &a, int es, int hw, int *warps, int *st
 template <typename T, int HW, int NP>
 int run_decode(const GroupedArgs &a, int *err, cudaStream_t s) {
     int warps = 0, stages = 0;
-    const DecodeSmem L = decode_plan(a, (int)sizeof(T), HW, &warps, &stages);
+    const DecodeSmem L = decode_plan(a, (int)sizeof(T), HW, decode_threads(HW, NP), &warps, &stages);
     B200_REQUIRE(warps > 0, "grouped decode: head size too large");
     const int rep = a.heads / a.kv_heads, hg = (rep + GH - 1) / GH;
     int rc = allow_smem(grouped_decode_kernel<T, HW, NP>, L.bytes());
@@ -682,10 +988,25 @@ template <typename T, int HW>
 int run_decode_channels(const GroupedArgs &a, int *err, cudaStream_t s) {
     return a.vdim <= 64 ? run_decode<T, HW, 1>(a, err, s) : a.vdim <= 128 ? run_decode<T, HW, 2>(a, err, s) : run_decode<T, HW, 4>(a, err, s);
 }
-template <typename T>
-int run_decode_heads(const GroupedArgs &a, int *err, cudaStream_t s) {
+int run_decode_f32(const GroupedArgs &a, int *err, cudaStream_t s) {
     const int rep = a.heads / a.kv_heads;
-    return rep > 4 ? run_decode_channels<T, 8>(a, err, s) : rep > 2 ? run_decode_channels<T, 4>(a, err, s) : rep > 1 ? run_decode_channels<T, 2>(a, err, s) : run_decode_channels<T, 1>(a, err, s);
+    return rep > 4 ? run_decode_channels<float, 8>(a, err, s) : rep > 2 ? run_decode_channels<float, 4>(a, err, s) : rep > 1 ? run_decode_channels<float, 2>(a, err, s)
+                                                                                                              : run_decode_channels<float, 1>(a, err, s);
+}
+bool decode_mma_plan(const GroupedArgs &a, int *warps, int *stages) {
+    for (*warps = DW; *warps >= 1; *warps /= 2)
+        for (*stages = 2; *stages >= 1; --*stages)
+            if ((size_t)DecodeMmaSmem(a.dim, a.vdim, *warps, *stages).bytes <= SMEM_MAX) return true;
+    return false;
+}
+template <int NT>
+int run_decode_mma(const GroupedArgs &a, int warps, int stages, int *err, cudaStream_t s) {
+    const int rep = a.heads / a.kv_heads, hg = (rep + GH - 1) / GH;
+    const size_t smem = (size_t)DecodeMmaSmem(a.dim, a.vdim, warps, stages).bytes;
+    int rc = allow_smem(grouped_decode_mma_kernel<NT>, smem);
+    if (rc != B200_STATUS_SUCCESS) return rc;
+    return launch_pdl_cluster(grouped_decode_mma_kernel<NT>, dim3((unsigned)a.splits, (unsigned)(a.kv_heads * hg), (unsigned)a.n), dim3((unsigned)(32 * warps)),
+                              (unsigned)a.splits, smem, s, a, hg, stages, err);
 }
 template <typename T, typename Y>
 int run_any(const GroupedArgs &a, int *err, cudaStream_t s) {
@@ -739,12 +1060,14 @@ int launch_grouped_decode(const GroupedArgs &a, cudaStream_t s) {
     if (rc != B200_STATUS_SUCCESS || a.n == 0) return rc;
     B200_REQUIRE(a.cells && a.seg && a.row_seg && a.tab && a.y && a.n_seg > 0 && a.splits >= 1 && a.splits <= SPLITS_MAX, "grouped decode: bad operand");
     int warps = 0, stages = 0;
-    decode_plan(a, a.type == B200_TYPE_F32 ? 4 : 2, GH, &warps, &stages);
-    if (a.vdim > 256 || warps == 0) {   // heads a block cannot hold
+    if (a.type == B200_TYPE_F32) decode_plan(a, 4, GH, GT, &warps, &stages);
+    else if (!decode_mma_plan(a, &warps, &stages)) warps = 0;
+    if (a.vdim > 256 || warps == 0 || a.n_cells > 0x7fffffffLL) {   // heads a block cannot hold
         rc = launch_grouped_store(a, s);
         return rc != B200_STATUS_SUCCESS ? rc : launch_grouped_attn(a, s);
     }
-    return a.type == B200_TYPE_F32 ? run_decode_heads<float>(a, err, s) : run_decode_heads<__nv_bfloat16>(a, err, s);
+    if (a.type == B200_TYPE_F32) return run_decode_f32(a, err, s);
+    return a.vdim <= 64 ? run_decode_mma<4>(a, warps, stages, err, s) : a.vdim <= 128 ? run_decode_mma<8>(a, warps, stages, err, s) : run_decode_mma<16>(a, warps, stages, err, s);
 }
 
 }  // namespace b200
