@@ -93,7 +93,7 @@ int b200_llama_get_hparams(const b200_llama *ctx, struct b200_llama_hparams *out
 
 /* ---- models described by a configuration file --------------------------------------------------------------
  * Architectures other than llama come as a folder with config.json and model.safetensors; config.json's "architecture"
- * picks one of the library's (Rukusun).  dtype: what the weight matrices are kept in, B200_TYPE_BF16 (matrix products with
+ * picks one of the library's (Rukusun, Lenolix).  dtype: what the weight matrices are kept in, B200_TYPE_BF16 (matrix products with
  * BF16 operands and F32 sums; norms, recurrences, scores and the residual stream in F32) or B200_TYPE_F32 (everything in
  * F32).  n_seq: sequences alive at a time (state slots).  b200_model_load_dir loads the folder; b200_model_new makes the
  * context of a configuration (the text of a config.json) whose tensors b200_llama_set_tensor then sets under their names in the

@@ -88,37 +88,14 @@ grouped_store_kernel(GroupedArgs a, int *err) {
 }
 
 // ---- few rows ------------------------------------------------------------------------------------------------
-template <typename T>
-struct Piece;   // 16 bytes of a cell's row
-template <>
-struct Piece<__nv_bfloat16> {
-    static constexpr int E = 8;
-    static __device__ __forceinline__ void unpack(const uint4 &w, float (&f)[8]) {
-        f[0] = bf16_lo(w.x); f[1] = bf16_hi(w.x); f[2] = bf16_lo(w.y); f[3] = bf16_hi(w.y);
-        f[4] = bf16_lo(w.z); f[5] = bf16_hi(w.z); f[6] = bf16_lo(w.w); f[7] = bf16_hi(w.w);
-    }
-    static __device__ __forceinline__ float2 pair(const __nv_bfloat16 *p) {
-        const uint32_t w = *reinterpret_cast<const uint32_t *>(p);
-        return make_float2(bf16_lo(w), bf16_hi(w));
-    }
-};
-template <>
-struct Piece<float> {
-    static constexpr int E = 4;
-    static __device__ __forceinline__ void unpack(const uint4 &w, float (&f)[4]) {
-        f[0] = __uint_as_float(w.x); f[1] = __uint_as_float(w.y); f[2] = __uint_as_float(w.z); f[3] = __uint_as_float(w.w);
-    }
-    static __device__ __forceinline__ float2 pair(const float *p) { return *reinterpret_cast<const float2 *>(p); }
-};
-
 // shared memory of a block of nw warps: each warp's own tiles (when they are done, the warps' sums), then floats at the offsets
 struct DecodeSmem {
     int units, tile;                       // 16-byte units of an entry's row, bytes of a tile
     size_t tiles;                          // bytes of the part ahead of the floats
     int q, p, m, l, w, out, ml, floats;    // offsets
-    __host__ __device__ DecodeSmem(int dim, int vdim, int es, int hw, int nw, int stages) {
+    __host__ __device__ DecodeSmem(int dim, int vdim, int hw, int nw, int stages) {
         const int d = pad8(dim), e = pad8(vdim);
-        units = (d + e) * es / 16;
+        units = (d + e) / 4;
         while (units % 4 != 2) units++;    // the two lanes of four neighbouring entries meet eight different bank groups
         tile = GK * units * 16;
         const size_t sums = (size_t)nw * hw * e * 4;
@@ -166,17 +143,18 @@ __device__ __noinline__ void fresh_row(const float *k, const float *v, const flo
     }
 }
 
-// A warp owns a stretch of the entries from load to weighted sum (no barrier until the end): two lanes share an entry's scores, then a
+// F32 cells.  A warp owns a stretch of the entries from load to weighted sum (no barrier until the end): two lanes share an entry's scores, then a
 // lane owns NP pairs of value channels.
-template <typename T, int HW, int NP>
+template <int HW, int NP>
 __global__ void __launch_bounds__(decode_threads(HW, NP), 1)
 grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
-    constexpr int PE = Piece<T>::E;
+    typedef float T;
+    constexpr int PE = 4;   // elements of 16 bytes
     extern __shared__ __align__(16) uint8_t g_raw[];
     cg::cluster_group cluster = cg::this_cluster();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
     const int dim = pad8(a.dim), vdim = pad8(a.vdim), kp = dim / PE, vp = vdim / PE;
-    const DecodeSmem L(a.dim, a.vdim, (int)sizeof(T), HW, nw, stages);
+    const DecodeSmem L(a.dim, a.vdim, HW, nw, stages);
     float *f32 = (float *)(g_raw + L.tiles);
     float *sq = f32 + L.q, *sp = f32 + L.p + warp * GK * HW, *sm = f32 + L.m, *sl = f32 + L.l, *sw = f32 + L.w, *sout = f32 + L.out, *sml = f32 + L.ml;
     const int rep = a.heads / a.kv_heads, g = blockIdx.y / head_groups, hg = blockIdx.y % head_groups, h0 = hg * GH, nh = min(HW, rep - h0);
@@ -270,18 +248,14 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
             for (int h = 0; h < HW; h++) s[h] = 0.0f;
 #pragma unroll 2
             for (int p = part; p < kp; p += 2) {
-                float f[PE];
-                Piece<T>::unpack(*reinterpret_cast<const uint4 *>(kr + p * PE), f);
+                const float4 f = *reinterpret_cast<const float4 *>(kr + p * PE);
 #pragma unroll
                 for (int h = 0; h < HW; h++) {
-#pragma unroll
-                    for (int e = 0; e < PE; e += 4) {
-                        const float4 x = *reinterpret_cast<const float4 *>(sq + h * dim + p * PE + e);
-                        s[h] = fmaf(x.x, f[e], s[h]);
-                        s[h] = fmaf(x.y, f[e + 1], s[h]);
-                        s[h] = fmaf(x.z, f[e + 2], s[h]);
-                        s[h] = fmaf(x.w, f[e + 3], s[h]);
-                    }
+                    const float4 x = *reinterpret_cast<const float4 *>(sq + h * dim + p * PE);
+                    s[h] = fmaf(x.x, f.x, s[h]);
+                    s[h] = fmaf(x.y, f.y, s[h]);
+                    s[h] = fmaf(x.z, f.z, s[h]);
+                    s[h] = fmaf(x.w, f.w, s[h]);
                 }
             }
         }
@@ -314,7 +288,7 @@ grouped_decode_kernel(GroupedArgs a, int head_groups, int stages, int *err) {
 #pragma unroll
             for (int i = 0; i < NP; i++) {
                 if (2 * lane + 64 * i >= vdim) break;
-                const float2 v = Piece<T>::pair(vc + (size_t)k * L.units * PE + 64 * i);
+                const float2 v = *reinterpret_cast<const float2 *>(vc + (size_t)k * L.units * PE + 64 * i);
 #pragma unroll
                 for (int h = 0; h < HW; h++) {
                     acc[h][2 * i] = fmaf(w[h], v.x, acc[h][2 * i]);
@@ -423,11 +397,11 @@ __device__ __forceinline__ void bulk_copy(void *dst, const void *src, uint32_t b
                  : "memory");
 }
 __device__ __forceinline__ bool bulk_wait(uint32_t bar, uint32_t parity) {
-    for (int round = 0; round < 2; round++)
+    for (int attempt = 0; attempt < 2; attempt++)
         for (uint32_t it = 0; it < BULK_WAIT_LIMIT; it++) {
             uint32_t ok;
             asm volatile("{ .reg .pred p; mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-            if (ok) return round == 0;
+            if (ok) return attempt == 0;
         }
     return false;
 }
@@ -440,7 +414,7 @@ grouped_decode_mma_kernel(GroupedArgs a, int head_groups, int stages, int *err) 
     __shared__ uint64_t bars[DW][2];   // a warp's tiles
     cg::cluster_group cluster = cg::this_cluster();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5, blocks = (int)gridDim.x;
-    const int dim = pad8(a.dim), vdim = pad8(a.vdim), kp = dim / 8, vp = vdim / 8;
+    const int dim = pad8(a.dim), vdim = pad8(a.vdim);
     const DecodeMmaSmem L(a.dim, a.vdim, nw, stages);
     bf *sQ = (bf *)(g_raw + L.q);
     float *sm = (float *)(g_raw + L.m), *sl = (float *)(g_raw + L.l), *sw = (float *)(g_raw + L.w), *recv = (float *)(g_raw + L.recv);
@@ -964,34 +938,34 @@ int allow_smem(K kernel, size_t smem) {
 constexpr size_t SMEM_MAX = 220 * 1024;
 
 // warps and tiles per warp that fit, as many warps as possible; 0 warps: none do
-DecodeSmem decode_plan(const GroupedArgs &a, int es, int hw, int threads, int *warps, int *stages) {
+DecodeSmem decode_plan(const GroupedArgs &a, int hw, int threads, int *warps, int *stages) {
     for (*warps = threads / 32; *warps >= 1; *warps /= 2)
         for (*stages = 2; *stages >= 1; --*stages) {
-            const DecodeSmem L(a.dim, a.vdim, es, hw, *warps, *stages);
+            const DecodeSmem L(a.dim, a.vdim, hw, *warps, *stages);
             if (L.bytes() <= SMEM_MAX) return L;
         }
     *warps = 0;
-    return DecodeSmem(1, 1, es, hw, 1, 1);
+    return DecodeSmem(1, 1, hw, 1, 1);
 }
-template <typename T, int HW, int NP>
+template <int HW, int NP>
 int run_decode(const GroupedArgs &a, int *err, cudaStream_t s) {
     int warps = 0, stages = 0;
-    const DecodeSmem L = decode_plan(a, (int)sizeof(T), HW, decode_threads(HW, NP), &warps, &stages);
+    const DecodeSmem L = decode_plan(a, HW, decode_threads(HW, NP), &warps, &stages);
     B200_REQUIRE(warps > 0, "grouped decode: head size too large");
     const int rep = a.heads / a.kv_heads, hg = (rep + GH - 1) / GH;
-    int rc = allow_smem(grouped_decode_kernel<T, HW, NP>, L.bytes());
+    int rc = allow_smem(grouped_decode_kernel<HW, NP>, L.bytes());
     if (rc != B200_STATUS_SUCCESS) return rc;
-    return launch_pdl_cluster(grouped_decode_kernel<T, HW, NP>, dim3((unsigned)a.splits, (unsigned)(a.kv_heads * hg), (unsigned)a.n), dim3((unsigned)(32 * warps)),
+    return launch_pdl_cluster(grouped_decode_kernel<HW, NP>, dim3((unsigned)a.splits, (unsigned)(a.kv_heads * hg), (unsigned)a.n), dim3((unsigned)(32 * warps)),
                               (unsigned)a.splits, L.bytes(), s, a, hg, stages, err);
 }
-template <typename T, int HW>
+template <int HW>
 int run_decode_channels(const GroupedArgs &a, int *err, cudaStream_t s) {
-    return a.vdim <= 64 ? run_decode<T, HW, 1>(a, err, s) : a.vdim <= 128 ? run_decode<T, HW, 2>(a, err, s) : run_decode<T, HW, 4>(a, err, s);
+    return a.vdim <= 64 ? run_decode<HW, 1>(a, err, s) : a.vdim <= 128 ? run_decode<HW, 2>(a, err, s) : run_decode<HW, 4>(a, err, s);
 }
 int run_decode_f32(const GroupedArgs &a, int *err, cudaStream_t s) {
     const int rep = a.heads / a.kv_heads;
-    return rep > 4 ? run_decode_channels<float, 8>(a, err, s) : rep > 2 ? run_decode_channels<float, 4>(a, err, s) : rep > 1 ? run_decode_channels<float, 2>(a, err, s)
-                                                                                                              : run_decode_channels<float, 1>(a, err, s);
+    return rep > 4 ? run_decode_channels<8>(a, err, s) : rep > 2 ? run_decode_channels<4>(a, err, s) : rep > 1 ? run_decode_channels<2>(a, err, s)
+                                                                                                              : run_decode_channels<1>(a, err, s);
 }
 bool decode_mma_plan(const GroupedArgs &a, int *warps, int *stages) {
     for (*warps = DW; *warps >= 1; *warps /= 2)
@@ -1060,7 +1034,7 @@ int launch_grouped_decode(const GroupedArgs &a, cudaStream_t s) {
     if (rc != B200_STATUS_SUCCESS || a.n == 0) return rc;
     B200_REQUIRE(a.cells && a.seg && a.row_seg && a.tab && a.y && a.n_seg > 0 && a.splits >= 1 && a.splits <= SPLITS_MAX, "grouped decode: bad operand");
     int warps = 0, stages = 0;
-    if (a.type == B200_TYPE_F32) decode_plan(a, 4, GH, GT, &warps, &stages);
+    if (a.type == B200_TYPE_F32) decode_plan(a, GH, GT, &warps, &stages);
     else if (!decode_mma_plan(a, &warps, &stages)) warps = 0;
     if (a.vdim > 256 || warps == 0 || a.n_cells > 0x7fffffffLL) {   // heads a block cannot hold
         rc = launch_grouped_store(a, s);

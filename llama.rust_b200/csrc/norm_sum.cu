@@ -11,7 +11,7 @@ namespace {
 
 constexpr int NS_VEC = 2;   // pieces of four elements a thread of the vector form holds
 
-// sum over a block of whole warps, the same value in every thread; part: 33 floats of shared memory
+// sum over a block of whole warps, the same value in every thread; part: 32 floats of shared memory
 __device__ __forceinline__ float row_sum(float v, float *part) {
     v = warp_sum(v);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;

@@ -64,7 +64,7 @@ def rotate_halves(x, pos, rot):
 def visible(i, mask):
     """the positions token i sees: a window that ends with itself, and the sequence's first tokens"""
     if not mask:
-        return list(range(i + 1))
+        return range(i + 1)
     return [j for j in range(i + 1) if j < mask.get("keep_first", 0) or i - j < mask["size"]]
 
 
@@ -75,6 +75,8 @@ def attention(q, k, v, sink, scale, mask, pos0):
     out = np.empty((T, H, v.shape[2]), F)
     for t in range(T):
         js = visible(pos0 + t, mask)
+        if len(js) == js[-1] - js[0] + 1:
+            js = slice(js[0], js[-1] + 1)   # (the same positions, without a copy)
         for h in range(H):
             out[t, h] = softmax_with_sink(k[js, h // per] @ q[t, h] * scale, sink[h]) @ v[js, h // per]
     return out

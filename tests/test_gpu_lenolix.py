@@ -231,6 +231,21 @@ def test_window_edges_and_kept_tokens(ll, window, keep, dtype):
         check(feed(m, toks, cycle(max(1, edge - 2), 2, 2, 2, 9, 17), 2), want, f"short portions over the edge, needle at {at}")
 
 
+@BOTH
+def test_far_keys_without_a_mask(ll, dtype):
+    """thousands of keys per row: every block and warp of a row's attention goes through several tiles, the needle in any of them"""
+    cfg, w = M.needle(None, 0, heads=2, kv_heads=1)
+    for at in (0, 1517, 4430):
+        toks = [t % 59 for t in M.tokens(cfg, 4500, 88 + at)]
+        toks[at] = 59
+        want = Expected(cfg, w, toks, dtype)
+        if dtype == "float32":
+            other = plain(cfg, w).feed([t if i != at else 0 for i, t in enumerate(toks)])
+            assert M.error(other[-1:], want.rows[-1:]).max() > 0.05, "the needle must show"
+        m = model(ll, cfg, w, dtype, n_ctx=4608, n_batch=4400, n_seq=1)
+        check(feed(m, toks, cycle(4400, 1, 1, 7, 8, 1, 30, 5)), want, f"needle at {at}")
+
+
 def test_pairs_across_portions(ll):
     """a portion's first token is paired with the last one of the portion before, whatever ran in between"""
     cfg = M.config([M.layer(ff=0)])

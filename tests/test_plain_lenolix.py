@@ -41,7 +41,7 @@ def test_rotation_turns_halves_and_keeps_relative_angles():
 def test_visible_positions():
     m = {"size": 3, "keep_first": 2}
     assert [L.visible(i, m) for i in (0, 1, 3, 4, 6)] == [[0], [0, 1], [0, 1, 2, 3], [0, 1, 2, 3, 4], [0, 1, 4, 5, 6]]
-    assert L.visible(2, None) == [0, 1, 2] and L.visible(5, {"size": 1}) == [5]
+    assert list(L.visible(2, None)) == [0, 1, 2] and L.visible(5, {"size": 1}) == [5]
 
 
 @pytest.mark.parametrize("loop", [None, (0, 2, 2), (1, 2, 3)])
